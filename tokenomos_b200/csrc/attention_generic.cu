@@ -13,7 +13,8 @@
 // Options beyond the reference: `keep_first` (the first positions of a sequence stay visible
 // behind a window, at their true positions), `sink` (the softmax's denominator has one more
 // term, a key of score 0 without a value: p_j = exp(s_j) / (1 + sum exp(s_j))), values of
-// another size than the keys (Dv), cache rows wider than either (Dp).
+// another size than the keys (Dv), cache rows wider than either (Dp), a soft cap (s <- cap tanh(s / cap))
+// and after it a bias by distance, s <- s + bias[h][min(i - j, L - 1)] (a float32 [H, L] table).
 #include <math.h>
 
 #include "common.cuh"
@@ -32,7 +33,7 @@ attn_generic_kernel(const T* q, const T* kv_pool, T* out,
                     const int* block_table, int bt_stride,
                     const int* tile_tok0, const int* tile_ntok, int H,
                     int Hkv, int D, int Dv, int Dp, int P, int window, int keep_first, int sink,
-                    int round_p, float scale, int heads_per_chunk) {
+                    int round_p, float scale, float cap, const float* __restrict__ bias, int L, int heads_per_chunk) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float smem[];
@@ -76,6 +77,8 @@ attn_generic_kernel(const T* q, const T* kv_pool, T* out,
     const int r = tid >> 3;   // my row
     const int sub = tid & 7;  // my lane within the row
     const int my_pos = row_pos[r];
+    const float inv_cap = cap > 0.f ? 1.f / cap : 0.f;
+    const float* my_bias = bias != nullptr ? bias + (size_t)(kvh * G + g0 + (r < rows ? r % gh : 0)) * L : nullptr;
     // a sink is a key of score 0 and no value that every row sees: the running maximum and sum
     // start from it
     float m_i = sink ? 0.f : -INFINITY, l_i = sink ? 1.f : 0.f;
@@ -121,6 +124,8 @@ attn_generic_kernel(const T* q, const T* kv_pool, T* out,
             d *= scale;
             const bool visible = my_pos >= 0 && j <= j_end && j <= my_pos &&
                                  (window <= 0 || my_pos - j < window || j < keep_first);
+            if (cap > 0.f) d = cap * tanhf(d * inv_cap);
+            if (visible && my_bias != nullptr) d += my_bias[min(my_pos - j, L - 1)];
             s[jj] = visible ? d : -INFINITY;
             mx = fmaxf(mx, s[jj]);
         }
@@ -183,14 +188,15 @@ TK_API int tk_attn_generic(const void* q, const void* kv_pool, void* out, const 
                            const int* tok_seq, const int* block_table, int bt_stride,
                            const int* tile_tok0, const int* tile_ntok, int n_tiles,
                            int tokens_per_tile, int H, int Hkv, int D, int Dv, int Dp, int P, int window,
-                           int keep_first, int sink, int round_p, float scale, int dtype,
+                           int keep_first, int sink, int round_p, float scale, float cap, const float* bias, int L, int dtype,
                            cudaStream_t stream) {
     TK_CHECK_ARG(H > 0 && Hkv > 0 && H % Hkv == 0, "attention: %d query heads over %d KV heads", H, Hkv);
     TK_CHECK_ARG(D > 0 && D <= MAX_D, "attention: head_dim %d outside 1..%d", D, MAX_D);
     TK_CHECK_ARG(Dv > 0 && Dv <= MAX_D, "attention: value size %d outside 1..%d", Dv, MAX_D);
     TK_CHECK_ARG(Dp >= D && Dp >= Dv, "attention: cache rows of %d for heads of %d and %d", Dp, D, Dv);
     TK_CHECK_ARG(keep_first >= 0, "attention: %d kept first positions", keep_first);
-    TK_CHECK_ARG(P > 0 && n_tiles >= 0, "attention: bad page size or tile count");
+    TK_CHECK_ARG(P > 0 && n_tiles >= 0 && cap >= 0.f, "attention: bad page size, tile count or cap");
+    TK_CHECK_ARG(bias == nullptr || L > 0, "attention: a distance bias of %d columns", L);
     if (n_tiles == 0) return 0;
     const int G = H / Hkv;
     TK_CHECK_ARG(tokens_per_tile >= 1 && tokens_per_tile <= BM, "attention: %d tokens per tile", tokens_per_tile);
@@ -204,13 +210,13 @@ TK_API int tk_attn_generic(const void* q, const void* kv_pool, void* out, const 
         tk_launch(attn_generic_kernel<float>, dim3(grid), dim3(THREADS), smem, stream, 
             (const float*)q, (const float*)kv_pool, (float*)out, positions, tok_seq, block_table,
             bt_stride, tile_tok0, tile_ntok, H, Hkv, D, Dv, Dp, P, window, keep_first, sink, round_p,
-            scale, heads_per_chunk);
+            scale, cap, bias, L, heads_per_chunk);
     } else if (dtype == TK_BF16) {
         cudaFuncSetAttribute(attn_generic_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         tk_launch(attn_generic_kernel<__nv_bfloat16>, dim3(grid), dim3(THREADS), smem, stream, 
             (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv_pool, (__nv_bfloat16*)out, positions,
             tok_seq, block_table, bt_stride, tile_tok0, tile_ntok, H, Hkv, D, Dv, Dp, P, window,
-            keep_first, sink, round_p, scale, heads_per_chunk);
+            keep_first, sink, round_p, scale, cap, bias, L, heads_per_chunk);
     } else {
         TK_CHECK_ARG(false, "attention: unknown dtype %d", dtype);
     }

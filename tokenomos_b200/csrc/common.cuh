@@ -85,6 +85,15 @@ __device__ __forceinline__ float silu_as(float g) {
     return g / (1.0f + expf(-g));
 }
 
+// The tanh form of gelu, z / 2 (1 + tanh(y)) = z sigmoid(2 y) with y = sqrt(2 / pi) (z + 0.044715 z^3); 16-bit
+// storage takes the special-function unit, 32-bit storage the accurate exponential.
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_as(float z) {
+    const float y2 = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+    if constexpr (sizeof(T) == 2) return z * rcp_approx(1.0f + ex2_approx(y2 * TK_NEG_LOG2E));
+    return z / (1.0f + expf(-y2));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -75,7 +75,7 @@ struct Fuse {
     int64_t ldr;
     // EPI_SWIGLU with another activation (glu != 0): g = min(gate, limit), u = clamp(up, -limit,
     // limit) (limit <= 0: no clamp), out = g * sigmoid(alpha g) * (u + shift), from the 32-bit
-    // sums, rounded once
+    // sums, rounded once; glu 2: out = gelu_tanh(gate) * up instead (no clamp)
     int glu;
     float glu_limit, glu_alpha, glu_shift;
 };
@@ -327,6 +327,10 @@ gemm_skinny_kernel(const __nv_bfloat16* x, int64_t ldx,
                 gate += bias[n0 + j];
                 up += bias[n0 + 8 + j];
             }
+            if (fuse.glu == 2) {
+                out[(size_t)tok * ldo + n0 / 2 + j] = from_f<TO>(gelu_tanh_as<TO>(gate) * up);
+                continue;
+            }
             if (fuse.glu) {
                 if (fuse.glu_limit > 0.f) {
                     gate = fminf(gate, fuse.glu_limit);
@@ -458,6 +462,12 @@ TK_API int tk_gemm_skinny_glu(const void* x, int64_t ldx, const void* w, int64_t
                               float alpha, float shift, cudaStream_t stream) {
     return skinny_launch(x, ldx, w, ldw, bias, out, ldo, M, N, K, out_dtype, 1, 0.f, nullptr, 0, 1, limit, alpha, shift,
                          stream);
+}
+
+// The same with the tanh form of gelu: out [M, N / 2] = gelu_tanh(gate) * up.
+TK_API int tk_gemm_skinny_gelu(const void* x, int64_t ldx, const void* w, int64_t ldw, const float* bias, void* out,
+                               int64_t ldo, int M, int N, int K, int out_dtype, cudaStream_t stream) {
+    return skinny_launch(x, ldx, w, ldw, bias, out, ldo, M, N, K, out_dtype, 1, 0.f, nullptr, 0, 2, 0.f, 0.f, 0.f, stream);
 }
 
 // The in-projection of a gated short conv with the conv in its epilogue, for a step in which every

@@ -1,0 +1,582 @@
+// Linear memories: recurrent mixers whose state is a matrix S [D, V] per head (D key channels, V values), walked
+// in token order with S in registers. Everything here is 32-bit arithmetic; the storage type T is only what q, k, v
+// are read as. Two rules and three kinds of decay, each a template parameter:
+//
+//   additive:  S <- a S;  S <- S + k v^T;                               o = S^T q
+//   delta:     S <- a S;  u = beta (v - S^T k);  S <- S + k u^T;        o = S^T q
+//
+//   a fixed per head (a constant of the layer), a per head and token, or a per key channel and token; the last two
+//   are a = exp(-A[h] * softplus(z + bias)). beta = sigmoid(zb). With `unit`, k and q are first brought to unit
+//   length, x / sqrt(sum(x^2) + 1e-6); with `act`, q, k and v first pass silu; q is multiplied by q_scale.
+//   Head h reads the q/k head h / (H / K).
+//
+// Eight lanes own a column of S: lane r of them has the rows 32 i + 4 r .. + 3 (i < R / 4), so that the state
+// [H, V, D] and the staged rows of k, q and a are read 16 bytes a lane, 128 bytes a column. The read-out is formed
+// from the decayed state and the step that is about to be written, o = (aS)^T q + (k . q) u, so that both sums
+// over the rows, (aS)^T k and (aS)^T q, run side by side and only the first is on the path from token to token.
+//
+// A step continues from the stored S exactly where the step before left it, and a token's arithmetic is the same
+// wherever the request was cut; a sequence at position 0 starts from zeros whatever its state row holds.
+#include <math.h>
+
+#include "common.cuh"
+
+namespace {
+enum : int { TK_K_LINMEM = 13 };
+constexpr int LM_LANES = 8;      // lanes of a column
+constexpr int LM_COLS = 4;       // columns of a warp (times the columns per thread)
+constexpr int LM_TOK = 16;       // tokens of a stage
+constexpr int LM_PROD = 4;       // warps that stage the next tokens
+
+enum : int { LM_ADD = 0, LM_DELTA = 1 };
+enum : int { LM_FIXED = 0, LM_HEAD = 1, LM_CHANNEL = 2 };
+
+struct LinMem {
+    const void* qkv;
+    int64_t stride;
+    int q_off, k_off, v_off;
+    const float* zb;             // [T, >= H] (delta)
+    int64_t zb_stride;
+    const float* za;             // [T, >= H] or [T, >= H D]; the decay itself when `ready`
+    int64_t za_stride;
+    int ready;
+    const float* bias;           // [H] or [H D]
+    const float* A;              // [H]: exp(A_log), or the fixed decays
+    float* state;                // [slots, H, V, D]
+    const int* cu_seqlens;
+    const int* seq_ctx;
+    const int* seq_slot;
+    float* y;                    // [T, H V]
+    int H, K, D, V;
+    float q_scale;
+    int unit, act;
+};
+
+__device__ __forceinline__ float lm_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float lm_decay(float z, float A) { return expf(-A * (z > 20.f ? z : log1pf(expf(z)))); }
+
+// Two 32-bit multiply-adds in one instruction (sm_100's packed form), each half rounded as the scalar one.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)),
+          "l"(reinterpret_cast<unsigned long long&>(c)));
+    return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
+    return d;
+}
+__device__ __forceinline__ float2 two(float x) { return make_float2(x, x); }
+__device__ __forceinline__ float sum8(float v) {      // over the eight lanes of a column
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    v += __shfl_xor_sync(0xffffffffu, v, 4);
+    return v;
+}
+
+// A column's rows between registers and memory
+template <int R>
+__device__ __forceinline__ void lm_load(float2 (&S)[R / 2], const float* col, int r, int D, bool ok) {
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const int d = 32 * i + 4 * r;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (ok && d < D) {
+            if (D % 4 == 0) {
+                v = *reinterpret_cast<const float4*>(col + d);
+            } else {
+                v.x = col[d];
+                if (d + 1 < D) v.y = col[d + 1];
+                if (d + 2 < D) v.z = col[d + 2];
+                if (d + 3 < D) v.w = col[d + 3];
+            }
+        }
+        S[2 * i] = make_float2(v.x, v.y);
+        S[2 * i + 1] = make_float2(v.z, v.w);
+    }
+}
+template <int R>
+__device__ __forceinline__ void lm_store(const float2 (&S)[R / 2], float* col, int r, int D, bool ok) {
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const int d = 32 * i + 4 * r;
+        if (!ok || d >= D) continue;
+        if (D % 4 == 0) {
+            *reinterpret_cast<float4*>(col + d) = make_float4(S[2 * i].x, S[2 * i].y, S[2 * i + 1].x, S[2 * i + 1].y);
+        } else {
+            col[d] = S[2 * i].x;
+            if (d + 1 < D) col[d + 1] = S[2 * i].y;
+            if (d + 2 < D) col[d + 2] = S[2 * i + 1].x;
+            if (d + 3 < D) col[d + 3] = S[2 * i + 1].y;
+        }
+    }
+}
+
+// One token for one column: S moves on, the column's output comes back (on all eight lanes). k, q, a: this lane's
+// first row of the staged vectors.
+template <int R, int RULE, int DECAY>
+__device__ __forceinline__ float lm_step(float2 (&S)[R / 2], const float* k, const float* q, const float* ga, float a,
+                                         float v, float beta, float kq) {
+    float2 kk[R / 2];
+    float2 pk0 = two(0.f), pk1 = two(0.f), pq0 = two(0.f), pq1 = two(0.f);
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        const float4 k4 = *reinterpret_cast<const float4*>(k + 32 * i);
+        const float4 q4 = *reinterpret_cast<const float4*>(q + 32 * i);
+        kk[2 * i] = make_float2(k4.x, k4.y);
+        kk[2 * i + 1] = make_float2(k4.z, k4.w);
+        if constexpr (DECAY == LM_CHANNEL) {
+            const float4 g4 = *reinterpret_cast<const float4*>(ga + 32 * i);
+            S[2 * i] = mul2(S[2 * i], make_float2(g4.x, g4.y));
+            S[2 * i + 1] = mul2(S[2 * i + 1], make_float2(g4.z, g4.w));
+        }
+        if constexpr (RULE == LM_DELTA) {
+            pk0 = fma2(S[2 * i], kk[2 * i], pk0);
+            pk1 = fma2(S[2 * i + 1], kk[2 * i + 1], pk1);
+        }
+        pq0 = fma2(S[2 * i], make_float2(q4.x, q4.y), pq0);
+        pq1 = fma2(S[2 * i + 1], make_float2(q4.z, q4.w), pq1);
+    }
+    float u = v, o;
+    if constexpr (RULE == LM_DELTA) {
+        const float p = sum8((pk0.x + pk0.y) + (pk1.x + pk1.y));
+        u = beta * (DECAY == LM_CHANNEL ? v - p : fmaf(-a, p, v));
+    }
+#pragma unroll
+    for (int i = 0; i < R / 2; ++i) S[i] = fma2(kk[i], two(u), DECAY == LM_CHANNEL ? S[i] : mul2(two(a), S[i]));
+    o = sum8((pq0.x + pq0.y) + (pq1.x + pq1.y));
+    return fmaf(kq, u, DECAY == LM_CHANNEL ? o : a * o);
+}
+
+// A warp stages one token's k and q (unit length, silu, q_scale), k . q and the decay per channel. A lane holds the
+// elements lane + 32 j.
+template <typename T, int DPL>
+__device__ __forceinline__ void lm_fetch(const LinMem& m, int row, int h, int lane, float (&kv)[DPL], float (&qv)[DPL]) {
+    const T* src = (const T*)m.qkv + (size_t)row * m.stride;
+    const int kh = h / (m.H / m.K);
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+        const int d = lane + 32 * j;
+        kv[j] = d < m.D ? to_f<T>(src[m.k_off + kh * m.D + d]) : 0.f;
+        qv[j] = d < m.D ? to_f<T>(src[m.q_off + kh * m.D + d]) : 0.f;
+    }
+}
+template <int DPL>
+__device__ __forceinline__ void lm_shape(const LinMem& m, int lane, float (&kv)[DPL], float (&qv)[DPL], float* ks, float* qs,
+                                         float* kq) {
+    if (m.act) {
+#pragma unroll
+        for (int j = 0; j < DPL; ++j) {
+            kv[j] = lm_silu(kv[j]);
+            qv[j] = lm_silu(qv[j]);
+        }
+    }
+    float sk = 0.f, sq = 0.f, s = 0.f;
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+        sk = fmaf(kv[j], kv[j], sk);
+        sq = fmaf(qv[j], qv[j], sq);
+        s = fmaf(kv[j], qv[j], s);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        s += __shfl_xor_sync(0xffffffffu, s, o);
+    }
+    const float mk = m.unit ? 1.0f / sqrtf(sk + 1e-6f) : 1.0f;
+    const float mq = (m.unit ? 1.0f / sqrtf(sq + 1e-6f) : 1.0f) * m.q_scale;
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+        ks[lane + 32 * j] = kv[j] * mk;
+        qs[lane + 32 * j] = qv[j] * mq;
+    }
+    if (lane == 0) *kq = s * mk * mq;
+}
+template <int DPL>
+__device__ __forceinline__ void lm_channel_decay(const LinMem& m, int row, int h, int lane, float A, float* gs) {
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+        const int d = lane + 32 * j;
+        float g = 1.f;
+        if (d < m.D) {
+            const float z = m.za[(size_t)row * m.za_stride + h * m.D + d];
+            g = m.ready ? z : lm_decay(z + m.bias[h * m.D + d], A);
+        }
+        gs[d] = g;
+    }
+}
+}  // namespace
+
+// Portions: a block owns 4 `cw` columns of a head of a sequence, a column per eight lanes of its first cw warps. The
+// last LM_PROD warps stage the next 16 tokens in shared memory while the others walk the 16 before.
+template <typename T, int R, int RULE, int DECAY>
+__global__ void __launch_bounds__(32 * (8 + LM_PROD))
+linmem_scan_kernel(const LinMem m, int cw) {
+    constexpr int DPL = R / 4, DP = 8 * R;               // the key size, padded
+    constexpr int VEC = DECAY == LM_CHANNEL ? 3 : 2;     // staged vectors per token
+    constexpr int PER = LM_TOK / LM_PROD;                // tokens a staging warp brings per stage
+    extern __shared__ __align__(16) float smem[];        // [2][k | q | a][TOK][DP], then [2][TOK][cols] values
+    __shared__ float kq_s[2][LM_TOK], beta_s[2][LM_TOK], a_s[2][LM_TOK];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int s = blockIdx.z, h = blockIdx.y, cols = LM_COLS * cw, c0 = blockIdx.x * cols;
+    const int first = m.cu_seqlens[s], len = m.cu_seqlens[s + 1] - first;
+    if (len <= 0) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r = lane & 7, col = c0 + warp * LM_COLS + (lane >> 3);
+    const bool walker = warp < cw;
+    const float A = m.A[h];
+    float* vs = smem + 2 * VEC * LM_TOK * DP;
+    float* st = m.state + (((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[s]) * m.H + h) * m.V + col) * m.D;
+    float2 S[R / 2];
+
+    auto stage = [&](int t0, int b) {                    // by the staging warps
+        const int pw = warp - cw;
+        float* ks = smem + (size_t)(b * VEC + 0) * LM_TOK * DP;
+        float* qs = smem + (size_t)(b * VEC + 1) * LM_TOK * DP;
+        float kv[PER][DPL], qv[PER][DPL];
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int t = min(t0 + pw + i * LM_PROD, len - 1);
+            lm_fetch<T, DPL>(m, first + t, h, lane, kv[i], qv[i]);
+        }
+        // values of all tokens, a lane per column
+        for (int i = threadIdx.x - 32 * cw; i < LM_TOK * cols; i += 32 * LM_PROD) {
+            const int t = min(t0 + i / cols, len - 1), c = c0 + i % cols;
+            float v = c < m.V ? to_f<T>(((const T*)m.qkv)[(size_t)(first + t) * m.stride + m.v_off + h * m.V + c]) : 0.f;
+            vs[b * LM_TOK * cols + i] = m.act ? lm_silu(v) : v;
+        }
+        if (pw == 0 && lane < LM_TOK) {
+            const int row = first + min(t0 + lane, len - 1);
+            if constexpr (RULE == LM_DELTA) beta_s[b][lane] = 1.0f / (1.0f + expf(-m.zb[(size_t)row * m.zb_stride + h]));
+            if constexpr (DECAY == LM_HEAD) a_s[b][lane] = lm_decay(m.za[(size_t)row * m.za_stride + h] + m.bias[h], A);
+        }
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int tk = pw + i * LM_PROD;
+            lm_shape<DPL>(m, lane, kv[i], qv[i], ks + tk * DP, qs + tk * DP, &kq_s[b][tk]);
+            if constexpr (DECAY == LM_CHANNEL)
+                lm_channel_decay<DPL>(m, first + min(t0 + tk, len - 1), h, lane, A,
+                                      smem + (size_t)(b * VEC + 2) * LM_TOK * DP + tk * DP);
+        }
+    };
+
+    if (walker) lm_load<R>(S, st, r, m.D, col < m.V && m.seq_ctx[s] > 0);
+    else stage(0, 0);
+    __syncthreads();
+    for (int t0 = 0, b = 0; t0 < len; t0 += LM_TOK, b ^= 1) {
+        if (walker) {
+            const int nt = min(LM_TOK, len - t0);
+            const float* ks = smem + (size_t)(b * VEC + 0) * LM_TOK * DP + 4 * r;
+            const float* qs = smem + (size_t)(b * VEC + 1) * LM_TOK * DP + 4 * r;
+            const float* gs = smem + (size_t)(b * VEC + VEC - 1) * LM_TOK * DP + 4 * r;
+            const float* vt = vs + b * LM_TOK * cols + warp * LM_COLS + (lane >> 3);
+            auto walk = [&](int t) {
+                return lm_step<R, RULE, DECAY>(S, ks + t * DP, qs + t * DP, gs + t * DP,
+                                               DECAY == LM_FIXED ? A : DECAY == LM_HEAD ? a_s[b][t] : 0.f, vt[t * cols],
+                                               RULE == LM_DELTA ? beta_s[b][t] : 0.f, kq_s[b][t]);
+            };
+            if (nt == LM_TOK) {
+                float keep = 0.f;
+#pragma unroll 8
+                for (int t = 0; t < LM_TOK; ++t) {
+                    const float o = walk(t);
+                    if (r == (t & 7)) keep = o;
+                    if ((t & 7) == 7 && col < m.V)
+                        m.y[(size_t)(first + t0 + t - 7 + r) * m.H * m.V + h * m.V + col] = keep;
+                }
+            } else {
+                for (int t = 0; t < nt; ++t) {
+                    const float o = walk(t);
+                    if (r == 0 && col < m.V) m.y[(size_t)(first + t0 + t) * m.H * m.V + h * m.V + col] = o;
+                }
+            }
+        } else if (t0 + LM_TOK < len) {
+            stage(t0 + LM_TOK, b ^ 1);
+        }
+        __syncthreads();
+    }
+    if (walker) lm_store<R>(S, st, r, m.D, col < m.V);
+}
+
+// Steps of single tokens (a few a sequence at most): the state streams through, CPT columns a thread, so that many
+// bytes are in flight; the block's warps stage a token's vectors together.
+template <typename T, int R, int RULE, int DECAY, int CPT>
+__global__ void __launch_bounds__(256)
+linmem_token_kernel(const LinMem m) {
+    constexpr int DPL = R / 4, DP = 8 * R;
+    __shared__ __align__(16) float ks[DP], qs[DP], gs[DECAY == LM_CHANNEL ? DP : 4];
+    __shared__ float kq_s;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int s = blockIdx.z, h = blockIdx.y, c0 = (blockIdx.x * warps + warp) * LM_COLS * CPT + (lane >> 3);
+    const int first = m.cu_seqlens[s], len = m.cu_seqlens[s + 1] - first;
+    if (len <= 0) return;
+    const int r = lane & 7;
+    const float A = m.A[h];
+    const bool carried = m.seq_ctx[s] > 0;
+    float* st = m.state + ((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[s]) * m.H + h) * m.V * m.D;
+    float2 S[CPT][R / 2];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const int col = c0 + LM_COLS * c;
+        lm_load<R>(S[c], st + (size_t)col * m.D, r, m.D, carried && col < m.V);
+    }
+    for (int t = 0; t < len; ++t) {
+        const int row = first + t;
+        float v[CPT], beta = 0.f, a = A;
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+            const int col = c0 + LM_COLS * c;
+            v[c] = col < m.V ? to_f<T>(((const T*)m.qkv)[(size_t)row * m.stride + m.v_off + h * m.V + col]) : 0.f;
+            if (m.act) v[c] = lm_silu(v[c]);
+        }
+        if constexpr (RULE == LM_DELTA) beta = 1.0f / (1.0f + expf(-m.zb[(size_t)row * m.zb_stride + h]));
+        if constexpr (DECAY == LM_HEAD) a = lm_decay(m.za[(size_t)row * m.za_stride + h] + m.bias[h], A);
+        if (t > 0) __syncthreads();
+        if (warp == 0) {
+            float kv[DPL], qv[DPL];
+            lm_fetch<T, DPL>(m, row, h, lane, kv, qv);
+            lm_shape<DPL>(m, lane, kv, qv, ks, qs, &kq_s);
+        }
+        if constexpr (DECAY == LM_CHANNEL) {
+            for (int d = threadIdx.x; d < DP; d += blockDim.x) {
+                float g = 1.f;
+                if (d < m.D) {
+                    const float z = m.za[(size_t)row * m.za_stride + h * m.D + d];
+                    g = m.ready ? z : lm_decay(z + m.bias[h * m.D + d], A);
+                }
+                gs[d] = g;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+            const float o = lm_step<R, RULE, DECAY>(S[c], ks + 4 * r, qs + 4 * r, gs + (DECAY == LM_CHANNEL ? 4 * r : 0), a,
+                                                    v[c], beta, kq_s);
+            const int col = c0 + LM_COLS * c;
+            if (r == 0 && col < m.V) m.y[(size_t)row * m.H * m.V + h * m.V + col] = o;
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const int col = c0 + LM_COLS * c;
+        lm_store<R>(S[c], st + (size_t)col * m.D, r, m.D, col < m.V);
+    }
+}
+
+namespace {
+template <typename T, int R, int RULE, int DECAY>
+void lm_launch(const LinMem& m, int n_seqs, bool tokens, int sm_count, cudaStream_t stream) {
+    if (tokens) {
+        constexpr int CPT = R >= 32 ? 1 : 2;
+        const int per_warp = LM_COLS * CPT;
+        int warps = (m.V + per_warp - 1) / per_warp;
+        const int blocks = (warps + 7) / 8;
+        warps = (warps + blocks - 1) / blocks;
+        tk_launch(linmem_token_kernel<T, R, RULE, DECAY, CPT>, dim3(blocks, m.H, n_seqs), dim3(32 * warps), 0, stream, m);
+        return;
+    }
+    // as many columns a block as leave a block for every SM
+    int cw = 8;
+    while (cw > 2 && (m.V + LM_COLS * cw - 1) / (LM_COLS * cw) * m.H * n_seqs < sm_count) cw /= 2;
+    const int cols = LM_COLS * cw;
+    const size_t smem = (2 * (size_t)(DECAY == LM_CHANNEL ? 3 : 2) * LM_TOK * 8 * R + 2 * (size_t)LM_TOK * cols) * sizeof(float);
+    static size_t raised = 48 * 1024;
+    if (smem > raised) {
+        cudaFuncSetAttribute(linmem_scan_kernel<T, R, RULE, DECAY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        raised = smem;
+    }
+    tk_launch(linmem_scan_kernel<T, R, RULE, DECAY>, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * (cw + LM_PROD)),
+              smem, stream, m, cw);
+}
+
+template <typename T, int RULE, int DECAY>
+void lm_rows(const LinMem& m, int n_seqs, bool tokens, int sm_count, cudaStream_t stream) {
+    if (m.D <= 32) lm_launch<T, 4, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
+    else if (m.D <= 64) lm_launch<T, 8, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
+    else if (m.D <= 128) lm_launch<T, 16, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
+    else lm_launch<T, 32, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
+}
+}  // namespace
+
+TK_API int tk_linmem_max_dim() { return 256; }
+
+// qkv: [T, >= ...] rows `stride` apart holding q (K x D) at column q_off, k at k_off, v (H x V) at v_off; rule 0
+// additive, 1 delta (zb: float32 [T, >= H] rows zb_stride apart, beta's logits); decay 0 fixed (A: float32 [H], the
+// decays), 1 per head, 2 per channel (za: float32 [T, >= H] or [T, >= H D] rows za_stride apart, bias likewise one
+// row, A: float32 [H]); ready: za holds the decays themselves. state: float32 [slots, H, V, D]; y: float32 [T, H V].
+TK_API int tk_linmem_scan(const void* qkv, int64_t stride, int q_off, int k_off, int v_off, int rule, const float* zb,
+                          int64_t zb_stride, int decay, const float* za, int64_t za_stride, int ready, const float* bias,
+                          const float* A, float* state, const int* cu_seqlens, const int* seq_ctx, const int* seq_slot,
+                          int n_seqs, int tokens, float* y, int H, int K, int D, int V, float q_scale, int unit, int act,
+                          int sm_count, int dtype, cudaStream_t stream) {
+    TK_CHECK_ARG(H > 0 && K > 0 && H % K == 0 && D > 0 && V > 0, "linear memory: %d heads over %d q/k heads", H, K);
+    TK_CHECK_ARG(D <= tk_linmem_max_dim(), "linear memory: a key size of %d; up to %d are built", D, tk_linmem_max_dim());
+    TK_CHECK_ARG((rule == LM_ADD && decay == LM_FIXED) || (rule == LM_DELTA && (decay == LM_HEAD || decay == LM_CHANNEL)),
+                 "linear memory: rule %d with decay %d is not built", rule, decay);
+    TK_CHECK_ARG(rule == LM_ADD || (zb != nullptr && za != nullptr && bias != nullptr), "linear memory: missing gates");
+    TK_CHECK_ARG(n_seqs >= 0 && tokens >= 0 && A != nullptr, "linear memory: bad sizes");
+    if (n_seqs == 0) return 0;
+    const LinMem m{qkv, stride, q_off, k_off, v_off, zb, zb_stride, za, za_stride, ready, bias, A, state, cu_seqlens, seq_ctx,
+                   seq_slot, y, H, K, D, V, q_scale, unit, act};
+    const bool few = tokens < 4 * n_seqs;      // single tokens, not portions
+#define TK_LM(TT)                                                                       \
+    do {                                                                                \
+        if (rule == LM_ADD) lm_rows<TT, LM_ADD, LM_FIXED>(m, n_seqs, few, sm_count, stream);          \
+        else if (decay == LM_HEAD) lm_rows<TT, LM_DELTA, LM_HEAD>(m, n_seqs, few, sm_count, stream);  \
+        else lm_rows<TT, LM_DELTA, LM_CHANNEL>(m, n_seqs, few, sm_count, stream);                     \
+    } while (0)
+    if (dtype == TK_F32) TK_LM(float);
+    else if (dtype == TK_BF16) TK_LM(__nv_bfloat16);
+    else TK_CHECK_ARG(false, "linear memory: unknown dtype %d", dtype);
+#undef TK_LM
+    TK_CHECK_LAUNCH("linmem_scan");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// out = group_norm(y) * w * gate(z): y's row in `groups` equal parts, each divided by its own
+// sqrt(mean + eps); gate silu or sigmoid. One warp per (row, group), or, for parts longer than
+// LM_WARP_PART, one block.
+// ---------------------------------------------------------------------------------------------
+namespace {
+constexpr int LM_WARP_PART = 512;
+enum : int { LM_GATE_SILU = 0, LM_GATE_SIGMOID = 1 };
+
+// 16-bit storage takes the special-function unit's exponential and reciprocal (a few ulp of a float, far below the
+// one rounding that follows), 32-bit storage the accurate functions
+template <typename T>
+__device__ __forceinline__ float lm_gate(float z, int kind) {
+    float s;
+    if constexpr (sizeof(T) == 2) s = rcp_approx(1.0f + ex2_approx(z * TK_NEG_LOG2E));
+    else s = 1.0f / (1.0f + expf(-z));
+    return kind == LM_GATE_SILU ? z * s : s;
+}
+}  // namespace
+
+template <typename T, int ITEMS, bool BLOCK>
+__global__ void __launch_bounds__(256)
+norm_gate_kernel(const float* y, const T* z, int64_t z_stride, const float* __restrict__ w, float eps, T* out, int rows,
+                 int width, int groups, int kind) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int unit = BLOCK ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int lane = BLOCK ? threadIdx.x : (threadIdx.x & 31), step = BLOCK ? 256 : 32;
+    if (!BLOCK && unit >= rows * groups) return;
+    const int r = unit / groups, gw = width / groups, c0 = (unit % groups) * gw;
+    const float* src = y + (size_t)r * width + c0;
+    const T* gate = z + (size_t)r * z_stride + c0;
+    T* dst = out + (size_t)r * width + c0;
+    float keep[ITEMS], zv[ITEMS], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = lane + step * k;
+        keep[k] = i < gw ? src[i] : 0.f;
+        zv[k] = i < gw ? to_f<T>(gate[i]) : 0.f;
+        ss = fmaf(keep[k], keep[k], ss);
+    }
+    for (int i = lane + step * ITEMS; i < gw; i += step) ss = fmaf(src[i], src[i], ss);
+    ss = BLOCK ? block_sum(ss, red) : warp_sum(ss);
+    const float rstd = 1.0f / sqrtf(ss / (float)gw + eps);
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = lane + step * k;
+        if (i < gw) dst[i] = from_f<T>(keep[k] * rstd * w[c0 + i] * lm_gate<T>(zv[k], kind));
+    }
+    for (int i = lane + step * ITEMS; i < gw; i += step)
+        dst[i] = from_f<T>(src[i] * rstd * w[c0 + i] * lm_gate<T>(to_f<T>(gate[i]), kind));
+}
+
+// y: float32 [rows, width]; z: [rows, width] (type dtype) rows `z_stride` apart; w: float32 [width]; out: [rows, width].
+TK_API int tk_norm_gate(const float* y, const void* z, int64_t z_stride, const float* w, float eps, void* out, int rows,
+                        int width, int groups, int kind, int dtype, cudaStream_t stream) {
+    TK_CHECK_ARG(rows >= 0 && width > 0 && groups > 0 && width % groups == 0, "norm and gate: a row of %d in %d groups",
+                 width, groups);
+    TK_CHECK_ARG(kind == LM_GATE_SILU || kind == LM_GATE_SIGMOID, "norm and gate: unknown gate %d", kind);
+    if (rows == 0) return 0;
+    const int gw = width / groups;
+#define TK_NG(TT, ITEMS, BLOCK)                                                                                      \
+    tk_launch(norm_gate_kernel<TT, ITEMS, BLOCK>, dim3(BLOCK ? rows * groups : (rows * groups + 7) / 8), dim3(256), 0, \
+              stream, y, (const TT*)z, z_stride, w, eps, (TT*)out, rows, width, groups, kind)
+#define TK_NG_T(TT)                                       \
+    do {                                                  \
+        if (gw > LM_WARP_PART) TK_NG(TT, 8, true);        \
+        else if (gw > 128) TK_NG(TT, 16, false);          \
+        else TK_NG(TT, 4, false);                         \
+    } while (0)
+    if (dtype == TK_F32) TK_NG_T(float);
+    else if (dtype == TK_BF16) TK_NG_T(__nv_bfloat16);
+    else TK_CHECK_ARG(false, "norm and gate: unknown dtype %d", dtype);
+#undef TK_NG_T
+#undef TK_NG
+    TK_CHECK_LAUNCH("norm_gate");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// Two mixers' outputs joined: out = coef * (a / rms(a) * wa + b / rms(b) * wb), rms over the row with
+// eps inside the root, in 32-bit with one rounding. One block per row.
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+pair_norm_mean_kernel(const T* a, int64_t a_stride, const T* b, int64_t b_stride, const float* __restrict__ wa,
+                      const float* __restrict__ wb, float eps, float coef, T* out, int width) {
+    constexpr int ITEMS = 8;
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t r = blockIdx.x;
+    const T* pa = a + r * a_stride;
+    const T* pb = b + r * b_stride;
+    float va[ITEMS], vb[ITEMS], sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+        va[k] = i < width ? to_f<T>(pa[i]) : 0.f;
+        vb[k] = i < width ? to_f<T>(pb[i]) : 0.f;
+        sa = fmaf(va[k], va[k], sa);
+        sb = fmaf(vb[k], vb[k], sb);
+    }
+    for (int i = threadIdx.x + ITEMS * blockDim.x; i < width; i += blockDim.x) {
+        const float x = to_f<T>(pa[i]), y = to_f<T>(pb[i]);
+        sa = fmaf(x, x, sa);
+        sb = fmaf(y, y, sb);
+    }
+    const float ra = coef / sqrtf(block_sum(sa, red) / (float)width + eps);
+    const float rb = coef / sqrtf(block_sum(sb, red) / (float)width + eps);
+#pragma unroll
+    for (int k = 0; k < ITEMS; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (i < width) out[r * width + i] = from_f<T>(va[k] * ra * wa[i] + vb[k] * rb * wb[i]);
+    }
+    for (int i = threadIdx.x + ITEMS * blockDim.x; i < width; i += blockDim.x)
+        out[r * width + i] = from_f<T>(to_f<T>(pa[i]) * ra * wa[i] + to_f<T>(pb[i]) * rb * wb[i]);
+}
+
+// a, b: [rows, width] (type dtype) rows `a_stride` / `b_stride` apart; wa, wb: float32 [width]; out: [rows, width].
+TK_API int tk_pair_norm_mean(const void* a, int64_t a_stride, const void* b, int64_t b_stride, const float* wa,
+                             const float* wb, float eps, float coef, void* out, int rows, int width, int dtype,
+                             cudaStream_t stream) {
+    TK_CHECK_ARG(rows >= 0 && width > 0, "pair_norm_mean: bad sizes rows=%d width=%d", rows, width);
+    if (rows == 0) return 0;
+    const int threads = width >= 1024 ? 256 : 128;
+    if (dtype == TK_F32)
+        tk_launch(pair_norm_mean_kernel<float>, dim3(rows), dim3(threads), 0, stream, (const float*)a, a_stride,
+                  (const float*)b, b_stride, wa, wb, eps, coef, (float*)out, width);
+    else if (dtype == TK_BF16)
+        tk_launch(pair_norm_mean_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, (const __nv_bfloat16*)a,
+                  a_stride, (const __nv_bfloat16*)b, b_stride, wa, wb, eps, coef, (__nv_bfloat16*)out, width);
+    else
+        TK_CHECK_ARG(false, "pair_norm_mean: unknown dtype %d", dtype);
+    TK_CHECK_LAUNCH("pair_norm_mean");
+    return 0;
+}

@@ -291,6 +291,73 @@ TK_API int tk_glu_clamped(const void* gu, void* out, int rows, int inter, int bl
 }
 
 // ---------------------------------------------------------------------------------------------
+// gated activation with the tanh form of gelu: out = gelu_tanh(gate) * up; gu as for the clamped one
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void glu_gelu_kernel(const T* gu, T* out, int inter, int block) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const T* row = gu + t * 2 * inter;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < inter; c += gridDim.y * blockDim.x) {
+        const int gi = block > 0 ? (c / block) * 2 * block + c % block : c;
+        out[t * inter + c] = from_f<T>(gelu_tanh_as<T>(to_f<T>(row[gi])) * to_f<T>(row[block > 0 ? gi + block : inter + c]));
+    }
+}
+
+// 16 bytes of gate and of up per thread (bfloat16, inter % 8 == 0)
+__global__ void __launch_bounds__(256)
+glu_gelu_vec_kernel(const __nv_bfloat16* gu, __nv_bfloat16* out, int inter, int block) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const __nv_bfloat16* row = gu + t * 2 * inter;
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < inter; c += gridDim.y * blockDim.x * 8) {
+        const int gi = block > 0 ? (c / block) * 2 * block + c % block : c;
+        const uint4 graw = *reinterpret_cast<const uint4*>(row + gi);
+        const uint4 uraw = *reinterpret_cast<const uint4*>(row + (block > 0 ? gi + block : inter + c));
+        const uint32_t* g2 = reinterpret_cast<const uint32_t*>(&graw);
+        const uint32_t* u2 = reinterpret_cast<const uint32_t*>(&uraw);
+        uint4 packed;
+        uint32_t* o2 = reinterpret_cast<uint32_t*>(&packed);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float a = gelu_tanh_as<__nv_bfloat16>(__uint_as_float(g2[e] << 16)) * __uint_as_float(u2[e] << 16);
+            const float b = gelu_tanh_as<__nv_bfloat16>(__uint_as_float(g2[e] & 0xffff0000u)) *
+                            __uint_as_float(u2[e] & 0xffff0000u);
+            const __nv_bfloat162 r = __floats2bfloat162_rn(a, b);
+            o2[e] = *reinterpret_cast<const uint32_t*>(&r);
+        }
+        *reinterpret_cast<uint4*>(out + t * inter + c) = packed;
+    }
+}
+
+TK_API int tk_glu_gelu(const void* gu, void* out, int rows, int inter, int block, int dtype, cudaStream_t stream) {
+    TK_CHECK_ARG(rows >= 0 && inter > 0, "glu_gelu: bad sizes rows=%d inter=%d", rows, inter);
+    TK_CHECK_ARG(block >= 0 && (block == 0 || inter % block == 0), "glu_gelu: runs of %d channels do not divide %d", block,
+                 inter);
+    if (rows == 0) return 0;
+    const int threads = 256;
+    const dim3 grid(rows, min(ceil_div(inter, threads), 64));
+    if (dtype == TK_BF16 && inter % 8 == 0 && (block == 0 || block % 8 == 0) && (uintptr_t)gu % 16 == 0 &&
+        (uintptr_t)out % 16 == 0) {
+        tk_launch(glu_gelu_vec_kernel, dim3(rows, min(ceil_div(inter, threads * 8), 64)), dim3(threads), 0, stream,
+                  (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, inter, block);
+        TK_CHECK_LAUNCH("glu_gelu_vec");
+        return 0;
+    }
+    if (dtype == TK_F32)
+        tk_launch(glu_gelu_kernel<float>, grid, dim3(threads), 0, stream, (const float*)gu, (float*)out, inter, block);
+    else if (dtype == TK_BF16)
+        tk_launch(glu_gelu_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, (const __nv_bfloat16*)gu,
+                  (__nv_bfloat16*)out, inter, block);
+    else
+        TK_CHECK_ARG(false, "glu_gelu: unknown dtype %d", dtype);
+    TK_CHECK_LAUNCH("glu_gelu");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
 // element-wise sigmoid gate, in place: x[t, c] = T(x[t, c] * sigmoid(g[t, c])); g's rows may be
 // `ldg` elements apart (a column block of a wider projection's output)
 // ---------------------------------------------------------------------------------------------
@@ -474,5 +541,117 @@ TK_API int tk_stream32_group_norm(const float* stream_in, const void* x, int64_t
     else
         TK_CHECK_ARG(false, "stream32_group_norm: unknown dtype %d", dtype);
     TK_CHECK_LAUNCH("stream32_group_norm");
+    return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// The stream's add behind a norm of what is added, with the norm that reads the stream next:
+//   stream' = stream + x / sqrt(mean(x^2) + eps_x) * wx        (stream optional: zeros)
+//   y = T(stream' / sqrt(mean(stream'^2) + eps) * w)           (w optional: only the add)
+// wx carries whatever multiplies the normed rows (a residual factor). One block per row; the row stays in registers
+// where it is short enough (ITEMS steps of 4 elements with VEC, of one without), else x and the stream's own writes
+// are read again.
+// ---------------------------------------------------------------------------------------------
+template <typename T, int ITEMS, bool VEC>
+__global__ void __launch_bounds__(256)
+stream32_post_norm_kernel(const float* stream_in, const T* x, int64_t x_stride, const float* __restrict__ wx, float eps_x,
+                          const float* __restrict__ w, float eps, float* stream_out, T* y, int width) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float red[33];
+    const size_t r = blockIdx.x;
+    const float inv_w = 1.0f / (float)width;
+    if constexpr (VEC) {
+        float4 a[ITEMS], b[ITEMS];
+        float sx = 0.f;
+#pragma unroll
+        for (int k = 0; k < ITEMS; ++k) {
+            const int i = (threadIdx.x + k * blockDim.x) * 4;
+            a[k] = b[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < width) {
+                if (stream_in != nullptr) a[k] = *reinterpret_cast<const float4*>(stream_in + r * width + i);
+                b[k] = Quad<T>::load(x + r * x_stride + i);
+            }
+            sx += b[k].x * b[k].x + b[k].y * b[k].y + b[k].z * b[k].z + b[k].w * b[k].w;
+        }
+        const float rx = 1.0f / sqrtf(block_sum(sx, red) * inv_w + eps_x);
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < ITEMS; ++k) {
+            const int i = (threadIdx.x + k * blockDim.x) * 4;
+            if (i < width) {
+                const float4 g = *reinterpret_cast<const float4*>(wx + i);
+                a[k] = make_float4(fmaf(b[k].x * rx, g.x, a[k].x), fmaf(b[k].y * rx, g.y, a[k].y),
+                                   fmaf(b[k].z * rx, g.z, a[k].z), fmaf(b[k].w * rx, g.w, a[k].w));
+                *reinterpret_cast<float4*>(stream_out + r * width + i) = a[k];
+            }
+            ss += a[k].x * a[k].x + a[k].y * a[k].y + a[k].z * a[k].z + a[k].w * a[k].w;
+        }
+        if (w == nullptr) return;
+        const float rstd = 1.0f / sqrtf(block_sum(ss, red) * inv_w + eps);
+#pragma unroll
+        for (int k = 0; k < ITEMS; ++k) {
+            const int i = (threadIdx.x + k * blockDim.x) * 4;
+            if (i < width) {
+                const float4 g = *reinterpret_cast<const float4*>(w + i);
+                Quad<T>::store(y + r * width + i, make_float4(a[k].x * rstd * g.x, a[k].y * rstd * g.y, a[k].z * rstd * g.z,
+                                                              a[k].w * rstd * g.w));
+            }
+        }
+    } else {
+        float sx = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            const float v = to_f<T>(x[r * x_stride + i]);
+            sx = fmaf(v, v, sx);
+        }
+        const float rx = 1.0f / sqrtf(block_sum(sx, red) * inv_w + eps_x);
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            const float v = fmaf(to_f<T>(x[r * x_stride + i]) * rx, wx[i], stream_in != nullptr ? stream_in[r * width + i] : 0.f);
+            stream_out[r * width + i] = v;
+            ss = fmaf(v, v, ss);
+        }
+        if (w == nullptr) return;
+        const float rstd = 1.0f / sqrtf(block_sum(ss, red) * inv_w + eps);
+        for (int i = threadIdx.x; i < width; i += blockDim.x)
+            y[r * width + i] = from_f<T>(stream_out[r * width + i] * rstd * w[i]);
+    }
+}
+
+template <typename T>
+static void launch_post_norm(const float* stream_in, const void* x, int64_t x_stride, const float* wx, float eps_x,
+                             const float* w, float eps, float* stream_out, void* y, int rows, int width,
+                             cudaStream_t stream) {
+    const int threads = width >= 1024 ? 256 : 128;
+    auto aligned = [](const void* p, int to) { return ((uintptr_t)p & (to - 1)) == 0; };
+    const int tb = sizeof(T) == 2 ? 8 : 16;
+    const bool vec = width % 4 == 0 && x_stride % 4 == 0 && aligned(stream_in, 16) && aligned(stream_out, 16) &&
+                     aligned(wx, 16) && aligned(w, 16) && aligned(x, tb) && aligned(y, tb);
+#define TK_PN(ITEMS, VEC)                                                                                              \
+    tk_launch(stream32_post_norm_kernel<T, ITEMS, VEC>, dim3(rows), dim3(threads), 0, stream, stream_in, (const T*)x, \
+              x_stride, wx, eps_x, w, eps, stream_out, (T*)y, width)
+    if (vec && width <= 4 * threads) TK_PN(1, true);
+    else if (vec && width <= 8 * threads) TK_PN(2, true);
+    else if (vec && width <= 24 * threads) TK_PN(6, true);
+    else TK_PN(1, false);
+#undef TK_PN
+}
+
+// stream_in / stream_out: float [rows, width] (may be the same buffer; stream_in may be null); x: T rows `x_stride`
+// elements apart; wx, w: float [width] (w null: the add alone, no y).
+TK_API int tk_stream32_post_norm(const float* stream_in, const void* x, int64_t x_stride, const float* wx, float eps_x,
+                                 const float* w, float eps, float* stream_out, void* y, int rows, int width, int dtype,
+                                 cudaStream_t stream) {
+    TK_CHECK_ARG(rows >= 0 && width > 0, "stream32_post_norm: bad sizes rows=%d width=%d", rows, width);
+    TK_CHECK_ARG(x != nullptr && wx != nullptr && stream_out != nullptr, "stream32_post_norm: nothing to add");
+    TK_CHECK_ARG(w == nullptr || y != nullptr, "stream32_post_norm: a norm weight without an output");
+    if (rows == 0) return 0;
+    if (dtype == TK_F32)
+        launch_post_norm<float>(stream_in, x, x_stride, wx, eps_x, w, eps, stream_out, y, rows, width, stream);
+    else if (dtype == TK_BF16)
+        launch_post_norm<__nv_bfloat16>(stream_in, x, x_stride, wx, eps_x, w, eps, stream_out, y, rows, width, stream);
+    else
+        TK_CHECK_ARG(false, "stream32_post_norm: unknown dtype %d", dtype);
+    TK_CHECK_LAUNCH("stream32_post_norm");
     return 0;
 }

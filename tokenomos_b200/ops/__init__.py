@@ -255,15 +255,16 @@ def attention(q: torch.Tensor, kv_pool: torch.Tensor, positions: torch.Tensor,
               tok_seq: torch.Tensor, block_table: torch.Tensor, tile_tok0: torch.Tensor,
               tile_ntok: torch.Tensor, tokens_per_tile: int, window: int | None,
               scale: float, keep_first: int = 0, sink: bool = False, v_dim: int | None = None,
-              round_p: bool = True) -> torch.Tensor:
+              round_p: bool = True, cap: float = 0.0, bias: torch.Tensor | None = None) -> torch.Tensor:
     """Causal (optionally windowed) attention of ``q`` [T, H, D] over the paged cache
     ``kv_pool`` [pages, 2, Hkv, P, Dp], which already holds this step's keys. Tiles name runs of
     at most ``tokens_per_tile`` tokens of one sequence. ``keep_first``: that many first positions
     of a sequence stay visible behind the window; ``sink``: one is added to the softmax's
     denominator; ``v_dim``: the values' size (default: the keys'; the cache rows hold at least
     both); ``round_p``: the weights are rounded to the storage type before they meet the values
-    (the 16-bit reference's rounding) instead of staying 32-bit. Returns [T, H, v_dim]."""
-    _cuda(q, kv_pool, positions, tok_seq, block_table, tile_tok0, tile_ntok)
+    (the 16-bit reference's rounding) instead of staying 32-bit; ``cap`` > 0: scores ``cap * tanh(s / cap)``;
+    ``bias`` float32 [H, L]: ``bias[h, min(i - j, L - 1)]`` joins the (capped) score. Returns [T, H, v_dim]."""
+    _cuda(q, kv_pool, positions, tok_seq, block_table, tile_tok0, tile_ntok, bias)
     T, H, D = q.shape
     _, two, Hkv, P, Dp = kv_pool.shape
     Dv = D if v_dim is None else int(v_dim)
@@ -274,9 +275,18 @@ def attention(q: torch.Tensor, kv_pool: torch.Tensor, positions: torch.Tensor,
               _ptr(_i32(tok_seq, "tok_seq")), _ptr(_i32(block_table, "block_table")),
               block_table.stride(0), _ptr(_i32(tile_tok0, "tile_tok0")),
               _ptr(_i32(tile_ntok, "tile_ntok")), tile_tok0.numel(), tokens_per_tile, H, Hkv, D, Dv, Dp, P,
-              int(window or 0), int(keep_first), int(bool(sink)), int(bool(round_p)), float(scale),
-              _dtype_code(q), _stream())
+              int(window or 0), int(keep_first), int(bool(sink)), int(bool(round_p)), float(scale), float(cap or 0.0),
+              *_bias_table(bias, H), _dtype_code(q), _stream())
     return out
+
+
+def _bias_table(bias: torch.Tensor | None, heads: int):
+    """(pointer, columns) of a bias by distance [heads, L], or (None, 0)."""
+    if bias is None:
+        return None, 0
+    if bias.dtype != torch.float32 or not bias.is_contiguous() or bias.dim() != 2 or bias.shape[0] != heads:
+        raise KernelError(f"attention: the distance bias is a contiguous float32 [{heads}, L] table")
+    return bias.data_ptr(), bias.shape[1]
 
 
 def rotary_write(qkv: torch.Tensor, kv_pool: torch.Tensor | None, freq: torch.Tensor, cs_mult: float,
@@ -366,6 +376,32 @@ def glu_clamped(gu: torch.Tensor, limit: float | None, alpha: float, shift: floa
     out = torch.empty(rows, inter, dtype=gu.dtype, device=gu.device)
     _lib.call("tk_glu_clamped", _ptr(gu), _ptr(out), rows, inter, int(block), float(limit or 0.0), float(alpha),
               float(shift), _dtype_code(gu), _stream())
+    return out
+
+
+def glu_gelu(gu: torch.Tensor, block: int = 0) -> torch.Tensor:
+    """``gelu_tanh(gate) * up`` for ``gu = [gate | up]`` of width ``2 I`` (``block`` > 0: gate and up alternate in
+    runs of ``block`` channels), formed in 32-bit and rounded once."""
+    _cuda(gu)
+    if not gu.is_contiguous() or gu.shape[1] % 2:
+        raise KernelError("glu_gelu: input must be contiguous with an even width")
+    rows, inter = gu.shape[0], gu.shape[1] // 2
+    out = torch.empty(rows, inter, dtype=gu.dtype, device=gu.device)
+    _lib.call("tk_glu_gelu", _ptr(gu), _ptr(out), rows, inter, int(block), _dtype_code(gu), _stream())
+    return out
+
+
+def gemm_skinny_gelu(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None) -> torch.Tensor:
+    """The gate/up product of at most 16 rows with ``gelu_tanh(gate) * up`` in its epilogue (rows of ``w`` and
+    ``bias`` as in ``gemm_skinny_glu``). Returns [M, N / 2]."""
+    _cuda(x, w, bias)
+    M, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K or N % 16 or not gemm_skinny_ok(x, w):
+        raise KernelError(f"gemm_skinny_gelu: x {tuple(x.shape)} against w {tuple(w.shape)}")
+    out = torch.empty(M, N // 2, dtype=x.dtype, device=x.device)
+    _lib.call("tk_gemm_skinny_gelu", _ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(_f32vec(bias, "bias", N)),
+              _ptr(out), out.stride(0), M, N, K, _dtype_code(out), _stream())
     return out
 
 
@@ -1498,3 +1534,157 @@ def stream32_group_norm(stream: torch.Tensor | None, x: torch.Tensor | None, gat
               gate.stride(0) if gate is not None else 0, _ptr(_f32vec(weight, "norm weight", width)), float(eps),
               _ptr(new), _ptr(y), rows, width, int(groups), F32 if out_dtype == torch.float32 else BF16, _stream())
     return y, new
+
+
+def stream32_post_norm(stream: torch.Tensor | None, x: torch.Tensor, post_weight: torch.Tensor, post_eps: float,
+                       weight: torch.Tensor | None, eps: float, in_place: bool = False):
+    """``stream' = stream + x / sqrt(mean(x^2) + post_eps) * post_weight`` in 32-bit (``stream`` None: zeros; the weight
+    carries whatever factor the normed rows get), ``y = rmsnorm(stream') * weight`` rounded once to ``x``'s type.
+    Returns ``(y, stream')``; ``y`` None without ``weight``. ``in_place``: ``stream`` is updated instead of copied."""
+    _cuda(stream, x, post_weight, weight)
+    rows, width = x.shape
+    if x.stride(1) != 1:
+        raise KernelError("stream32_post_norm: rows of x must be contiguous")
+    if stream is not None and (stream.dtype != torch.float32 or not stream.is_contiguous() or tuple(stream.shape) != (rows, width)):
+        raise KernelError("stream32_post_norm: the stream is a contiguous float32 [rows, width] tensor")
+    new = stream if (in_place and stream is not None) else torch.empty(rows, width, dtype=torch.float32, device=x.device)
+    y = torch.empty(rows, width, dtype=x.dtype, device=x.device) if weight is not None else None
+    _lib.call("tk_stream32_post_norm", _ptr(stream), _ptr(x), x.stride(0), _ptr(_f32vec(post_weight, "post-norm weight", width)),
+              float(post_eps), _ptr(_f32vec(weight, "norm weight", width)), float(eps), _ptr(new), _ptr(y), rows, width,
+              _dtype_code(x), _stream())
+    return y, new
+
+
+# ---- linear memories: additive and delta-rule recurrences over a matrix state ---------------------------
+
+LINMEM_MAX_DIM = 256
+LINMEM_RULES = {"add": 0, "delta": 1}
+LINMEM_DECAYS = {"fixed": 0, "head": 1, "channel": 2}
+GATE_KINDS = {"silu": 0, "sigmoid": 1}
+
+
+def linmem_scan(qkv: torch.Tensor, offsets: tuple, rule: str, decay: str, A: torch.Tensor, state: torch.Tensor,
+                cu_seqlens: torch.Tensor, seq_ctx: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, heads: int, kv_heads: int,
+                dim: int, v_dim: int, q_scale: float = 1.0, unit: bool = False, act: bool = False,
+                beta: torch.Tensor | None = None, gates: torch.Tensor | None = None, bias: torch.Tensor | None = None,
+                ready: bool = False, sm_count: int = 148) -> torch.Tensor:
+    """A matrix memory per head over a step's tokens: ``S <- a S``, then ``S <- S + k v^T`` (``rule`` "add") or ``u =
+    sigmoid(beta) (v - S^T k), S <- S + k u^T`` ("delta"), ``y = S^T q``. ``qkv`` [T, *]: q (``kv_heads`` x dim) at column
+    ``offsets[0]``, k at ``offsets[1]``, v (``heads`` x v_dim) at ``offsets[2]``; head h reads q/k head ``h / (heads /
+    kv_heads)``. ``decay``: "fixed" (``A`` float32 [heads] holds a), "head" or "channel" (``a = exp(-A[h] softplus(gates
+    + bias))`` with ``gates`` float32 [T, >= heads] or [T, >= heads dim]; ``ready``: ``gates`` holds a). ``act``: q, k
+    and v pass silu first; ``unit``: q and k are brought to unit length; q is multiplied by ``q_scale``. ``state`` float32
+    [slots, heads, v_dim, dim]. Returns ``y`` float32 [T, heads v_dim]."""
+    _cuda(qkv, A, state, beta, gates, bias)
+    T = qkv.shape[0]
+    if qkv.stride(1) != 1:
+        raise KernelError("linmem_scan: rows of q, k and v with contiguous columns")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, v_dim, dim) or not state.is_contiguous():
+        raise KernelError(f"linmem_scan: the state is float32 [slots, {heads}, {v_dim}, {dim}]")
+    cols = {"fixed": 0, "head": heads, "channel": heads * dim}[decay]
+    for name, t, need in (("beta", beta, heads if rule == "delta" else 0), ("gates", gates, cols)):
+        if need and (t is None or t.dtype != torch.float32 or t.stride(1) != 1 or t.shape[0] != T or t.shape[1] < need):
+            raise KernelError(f"linmem_scan: {name} is float32 [{T}, >= {need}] with contiguous columns")
+    y = torch.empty(T, heads * v_dim, dtype=torch.float32, device=qkv.device)
+    _lib.call("tk_linmem_scan", _ptr(qkv), qkv.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]), LINMEM_RULES[rule],
+              _ptr(beta), beta.stride(0) if beta is not None else 0, LINMEM_DECAYS[decay], _ptr(gates),
+              gates.stride(0) if gates is not None else 0, int(bool(ready)), _ptr(_f32vec(bias, "decay bias", cols)) if cols else None,
+              _ptr(_f32vec(A, "A", heads)), _ptr(state), _ptr(_i32(cu_seqlens, "cu_seqlens")), _ptr(_i32(seq_ctx, "seq_ctx")),
+              _ptr(_i32(seq_slot, "seq_slot")), int(n_seqs), T, _ptr(y), heads, kv_heads, dim, v_dim, float(q_scale),
+              int(bool(unit)), int(bool(act)), int(sm_count), _dtype_code(qkv), _stream())
+    return y
+
+
+def norm_gate(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, gate: str) -> torch.Tensor:
+    """Each of the row's ``groups`` equal parts of ``y`` (float32 [T, C]) divided by its own ``sqrt(mean + eps)``, times
+    ``weight`` [C], times ``gate(z)`` ("silu" or "sigmoid"; ``z`` [T, C] in the storage type, rows may be strided)."""
+    _cuda(y, z, weight)
+    T, C = y.shape
+    if y.dtype != torch.float32 or not y.is_contiguous() or z.stride(1) != 1 or tuple(z.shape) != (T, C):
+        raise KernelError("norm_gate: y float32 [T, C] contiguous, z [T, C] with contiguous columns")
+    out = torch.empty(T, C, dtype=z.dtype, device=y.device)
+    _lib.call("tk_norm_gate", _ptr(y), _ptr(z), z.stride(0), _ptr(_f32vec(weight, "norm weight", C)), float(eps), _ptr(out), T, C,
+              int(groups), GATE_KINDS[gate], _dtype_code(z), _stream())
+    return out
+
+
+def pair_norm_mean(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, eps: float,
+                   coef: float = 0.5) -> torch.Tensor:
+    """``coef * (rmsnorm(a) * wa + rmsnorm(b) * wb)`` over the row, in 32-bit with one rounding."""
+    _cuda(a, b, wa, wb)
+    rows, width = a.shape
+    if a.dtype != b.dtype or a.shape != b.shape or a.stride(1) != 1 or b.stride(1) != 1:
+        raise KernelError("pair_norm_mean: two [rows, width] tensors of one type with contiguous columns")
+    out = torch.empty(rows, width, dtype=a.dtype, device=a.device)
+    _lib.call("tk_pair_norm_mean", _ptr(a), a.stride(0), _ptr(b), b.stride(0), _ptr(_f32vec(wa, "norm weight", width)),
+              _ptr(_f32vec(wb, "norm weight", width)), float(eps), float(coef), _ptr(out), rows, width, _dtype_code(a), _stream())
+    return out
+
+
+# ---- softmax attention with a soft cap and a bias by distance -----------------------------------------------
+
+def qkv_row_norm_write(qkv: torch.Tensor, wq: torch.Tensor, wk: torch.Tensor | None, eps: float, positions: torch.Tensor,
+                       tok_seq: torch.Tensor, block_table: torch.Tensor | None, pool: torch.Tensor | None, heads: int,
+                       kv_heads: int, dim: int, v_dim: int) -> torch.Tensor:
+    """From rows ``[q | k | v]`` the queries [T, heads, dim] and, in ``pool`` [pages, 2, kv_heads, P, row] at each token's
+    position, the keys and values; a token's whole q row and whole k row are RMS-normed (all heads at once) and
+    multiplied by ``wq`` / ``wk``. ``pool`` None: queries only."""
+    _cuda(qkv, wq, wk, positions, tok_seq, block_table, pool)
+    T = qkv.shape[0]
+    need = heads * dim + (kv_heads * (dim + v_dim) if pool is not None else 0)
+    if qkv.stride(1) != 1 or qkv.shape[1] < need:
+        raise KernelError(f"qkv_row_norm_write: rows of at least {need} contiguous columns")
+    q = torch.empty(T, heads, dim, dtype=qkv.dtype, device=qkv.device)
+    P = dp = bt = 0
+    if pool is not None:
+        if (pool.dtype != qkv.dtype or not pool.is_contiguous() or pool.dim() != 5 or pool.shape[1] != 2
+                or pool.shape[2] != kv_heads):
+            raise KernelError(f"qkv_row_norm_write: the pool is {qkv.dtype} [pages, 2, {kv_heads}, P, row]")
+        P, dp, bt = pool.shape[3], pool.shape[4], _i32(block_table, "block_table").stride(0)
+    _lib.call("tk_qkv_row_norm_write", _ptr(qkv), qkv.stride(0), _ptr(_f32vec(wq, "q norm weight", heads * dim)),
+              _ptr(_f32vec(wk, "k norm weight", kv_heads * dim)), float(eps), _ptr(_i32(positions, "positions")),
+              _ptr(_i32(tok_seq, "tok_seq")), _ptr(block_table), bt, _ptr(q), _ptr(pool), T, heads, max(kv_heads, 1), dim, v_dim, P,
+              dp, _dtype_code(qkv), _stream())
+    return q
+
+
+def attention_biased_mma_supported(heads: int, kv_heads: int, head_dim: int, v_dim: int, row: int,
+                                   dtype: torch.dtype) -> bool:
+    """Whether ``attention_biased_mma`` takes the shape (bfloat16, sizes in multiples of 8 up to 128, at most 16 query
+    heads per key/value head)."""
+    return dtype == torch.bfloat16 and bool(_lib.call("tk_attn_biased_mma_supported", heads, kv_heads, head_dim, v_dim, row))
+
+
+def attention_biased_mma_tokens(heads: int, kv_heads: int) -> int:
+    """Tokens per tile ``attention_biased_mma`` expects for prompt portions."""
+    return _lib.call("tk_attn_biased_mma_tokens", heads, kv_heads)
+
+
+def attention_biased_mma(q: torch.Tensor, kv_pool: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,
+                         tok_seq: torch.Tensor, block_table: torch.Tensor, tile_tok0: torch.Tensor | None,
+                         tile_ntok: torch.Tensor | None, singles: torch.Tensor | None, n_single: int, nsplit: int,
+                         window: int | None, scale: float, cap: float = 0.0, bias: torch.Tensor | None = None,
+                         bounded: bool = False) -> None:
+    """Softmax attention with scores ``cap tanh(q.k scale / cap) + bias[h, min(i - j, L - 1)]`` on the tensor cores: the
+    tiles of prompt portions (``attention_biased_mma_tokens`` tokens each) and ``n_single`` single tokens (their rows
+    in ``singles``; None: rows 0 .. n_single - 1), each shared ``nsplit`` ways over its keys. ``q`` [T, H, D], ``out``
+    [T, H, Dv], ``kv_pool`` [pages, 2, Hkv, P, row]. ``bounded``: cap and bias keep every score, in base-2 logarithms,
+    well inside a float's exponents, so the softmax needs no running maximum."""
+    _cuda(q, kv_pool, out, positions, tok_seq, block_table, tile_tok0, tile_ntok, singles, bias)
+    T, H, D = q.shape
+    _, two, Hkv, P, Dp = kv_pool.shape
+    Dv = out.shape[2]
+    if (two != 2 or kv_pool.dtype != q.dtype or q.dtype != torch.bfloat16 or tuple(out.shape[:2]) != (T, H)
+            or not (q.is_contiguous() and kv_pool.is_contiguous() and out.is_contiguous())):
+        raise KernelError("attention_biased_mma: bfloat16 q [T, H, D], out [T, H, Dv] and cache [pages, 2, Hkv, P, row]")
+    n_tiles = tile_tok0.numel() if tile_tok0 is not None else 0
+    part_o = part_ml = None
+    if n_single and nsplit > 1:
+        part_o = torch.empty(nsplit * n_single * H * Dv, dtype=torch.float32, device=q.device)
+        part_ml = torch.empty(nsplit * n_single * H * 2, dtype=torch.float32, device=q.device)
+    _lib.call("tk_attn_biased_mma", _ptr(q), _ptr(kv_pool), _ptr(out), _ptr(_i32(positions, "positions")),
+              _ptr(_i32(tok_seq, "tok_seq")), _ptr(_i32(block_table, "block_table")), block_table.stride(0),
+              _ptr(_i32(tile_tok0, "tile_tok0")) if n_tiles else None, _ptr(_i32(tile_ntok, "tile_ntok")) if n_tiles else None,
+              n_tiles, _ptr(_i32(singles, "singles")) if singles is not None else None, int(n_single), int(nsplit), _ptr(part_o),
+              _ptr(part_ml), H, Hkv, D, Dv, Dp, P, int(window or 0), float(scale), float(cap or 0.0), *_bias_table(bias, H),
+              int(bool(bounded)), _stream())

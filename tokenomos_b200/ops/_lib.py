@@ -35,7 +35,7 @@ _SIGNATURES = {
     "tk_head_gate": [P, P, L, I, I, I, I, P],
     "tk_qk_norm_rope_write": [P, L, P, P, P, P, F, P, P, P, P, I, I, I, I, I, I, I, I, P],
     "tk_attn_generic_rows": [],
-    "tk_attn_generic": [P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P],
+    "tk_attn_generic": [P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P, I, I, P],
     "tk_rotary_write": [P, L, P, P, P, F, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P],
     "tk_stream32_add_norm": [P, P, L, P, P, P, F, P, P, P, I, I, I, P],
     "tk_glu_clamped": [P, P, I, I, I, F, F, F, I, P],
@@ -106,6 +106,17 @@ _SIGNATURES = {
     "tk_qkv_maps_write": [P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, P],
     "tk_diff_combine": [P, P, I, I, F, F, F, I, P],
     "tk_stream32_group_norm": [P, P, L, P, L, P, F, P, P, I, I, I, I, P],
+    "tk_stream32_post_norm": [P, P, L, P, F, P, F, P, P, I, I, I, P],
+    "tk_glu_gelu": [P, P, I, I, I, I, P],
+    "tk_gemm_skinny_gelu": [P, L, P, L, P, P, L, I, I, I, I, P],
+    "tk_linmem_max_dim": [],
+    "tk_linmem_scan": [P, L, I, I, I, I, P, L, I, P, L, I, P, P, P, P, P, P, I, I, P, I, I, I, I, F, I, I, I, I, P],
+    "tk_norm_gate": [P, P, L, P, F, P, I, I, I, I, I, P],
+    "tk_pair_norm_mean": [P, L, P, L, P, P, F, F, P, I, I, I, P],
+    "tk_attn_biased_mma_supported": [I, I, I, I, I],
+    "tk_attn_biased_mma_tokens": [I, I],
+    "tk_attn_biased_mma": [P, P, P, P, P, P, I, P, P, I, P, I, I, P, P, I, I, I, I, I, I, I, F, F, P, I, I, P],
+    "tk_qkv_row_norm_write": [P, L, P, P, F, P, P, P, I, P, P, I, I, I, I, I, I, I, I, P],
 }
 
 
@@ -157,7 +168,8 @@ _QUERIES = {"tk_check_device", "tk_built_for", "tk_set_pdl", "tk_checks_enabled"
             "tk_attn_prefill_tc_tokens", "tk_attn_prefill_tc_status", "tk_gemm_tc_status", "tk_sample_status",
             "tk_attn_latent_rows", "tk_attn_latent_max_rank", "tk_gemm_grouped_tile", "tk_attn_latent_mma_rows",
             "tk_attn_latent_mma_supported", "tk_attn_pointwise_rows", "tk_attn_pointwise_mma_supported",
-            "tk_attn_pointwise_mma_tokens", "tk_ssd_max_state", "tk_ssd_split"}
+            "tk_attn_pointwise_mma_tokens", "tk_ssd_max_state", "tk_ssd_split", "tk_linmem_max_dim",
+            "tk_attn_biased_mma_supported", "tk_attn_biased_mma_tokens"}
 
 
 _fns: dict = {}

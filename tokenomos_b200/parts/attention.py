@@ -18,12 +18,14 @@ key has the weight ``sigmoid(s + bias[h])`` of its own score, with an optional c
 a bias by distance ``- r1[h] ln(1 + r2[h] (i - j))`` and a query temperature ``1 + coef ln(floor((i + 1)
 / every) + 1)``; ``PointwiseWeights``); ``diff`` (differential attention, ``DiffMaps``: every head has two
 softmax maps over the same values, each with its own half of the query and of the key, joined as
-``a_1 - lambda a_2`` and brought to unit root mean square per head). A position part may keep state per request (a short
+``a_1 - lambda a_2`` and brought to unit root mean square per head); ``shape`` (``ScoreShape``: the scores' soft cap ``c tanh(s / c)`` and,
+after it, a learned bias by distance). A position part may keep state per request (a short
 convolution on q, k and v): it then has ``state_specs()`` and is called with the layer's ``call``.
 """
 
 from __future__ import annotations
 
+import math
 import os
 from dataclasses import dataclass
 
@@ -64,6 +66,34 @@ class DiffMaps:
     eps: float
 
 
+@dataclass(frozen=True)
+class ScoreShape:
+    """What happens to a softmax layer's scores after ``q . k * scale``: ``s <- cap tanh(s / cap)`` (``cap`` 0: nothing),
+    then ``s <- s + bias[h, min(i - j, L - 1)]`` (``bias`` float32 [heads, L], L covering every distance up to the
+    window or to where it no longer changes; None: nothing)."""
+
+    cap: float = 0.0
+    bias: torch.Tensor | None = None
+
+    @property
+    def bounded(self) -> bool:
+        """Whether the scores, in base-2 logarithms, span little enough of a float's exponents that a softmax over them
+        needs no running maximum: between ``-2 cap`` and 0 around the bias."""
+        if self.cap <= 0:
+            return False
+        reach = 0.0 if self.bias is None else float(self.bias.abs().max())
+        return (2.0 * self.cap + 2.0 * reach) / math.log(2.0) <= 100.0
+
+
+def distance_bucket(n: int, rows: int, far: float) -> int:
+    """The row of a ``rows``-row table of biases for distance ``n``: the first half one by one, the second half in equal
+    steps of the logarithm up to ``far``."""
+    half = rows / 2
+    if n < half:
+        return n
+    return min(rows - 1, int(half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half))))
+
+
 class Attention:
     def __init__(self, qkv: Linear, o: Linear, heads: int, kv_heads: int, head_dim: int, rope,
                  eps: float, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
@@ -72,7 +102,7 @@ class Attention:
                  gate_fused: bool = False, tuning: Tuning = DEFAULT_TUNING, sink: bool = False,
                  keep_first: int = 0, v_dim: int | None = None, v_is_k: bool = False,
                  gate_kind: str = "head", exact: bool = False, pointwise: PointwiseWeights | None = None,
-                 diff: DiffMaps | None = None):
+                 diff: DiffMaps | None = None, shape: ScoreShape | None = None):
         """``gate``: the per-head gate's projection as a part of its own; ``gate_fused``: its rows
         are the last of ``qkv``'s instead (after q, k, v, then zero rows up to a multiple of 8), so
         that one product yields both. With ``diff``, ``heads`` counts the maps (twice the output heads)
@@ -94,13 +124,21 @@ class Attention:
         self.sink, self.keep_first, self.v_dim, self.v_is_k = bool(sink), int(keep_first), v_dim, bool(v_is_k)
         self.gate_kind, self.exact = gate_kind, bool(exact)
         self.pointwise = pointwise
+        self.shape = shape
+        if shape is not None:
+            if pointwise is not None or diff is not None or sink or keep_first:
+                raise ValueError("attention: a cap and a distance bias on the scores go with a plain softmax over a window")
+            if shape.bias is not None and shape.bias.shape[0] != heads:
+                raise ValueError(f"attention: a distance bias of {shape.bias.shape[0]} rows for {heads} heads")
+            self.shape_bounded = shape.bounded          # (asked once: it reads the bias from the device)
         if pointwise is not None and (sink or keep_first):
             raise ValueError("attention: a sink and kept first positions belong to the softmax")
         # what the one-kernel decode form and the norms folded into the projections do not take
         # (the tensor-core kernels take all of it but a value size of its own; the general
         # kernel takes everything)
         self.extended = bool(self.sink or self.keep_first or self.v_is_k or v_dim != head_dim
-                             or gate_kind != "head" or self.exact or pointwise is not None or diff is not None)
+                             or gate_kind != "head" or self.exact or pointwise is not None or diff is not None
+                             or shape is not None)
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads over {kv_heads} KV heads")
         if head_dim > ops.ATTENTION_MAX_HEAD_DIM:
@@ -152,6 +190,19 @@ class Attention:
         if self.diff is not None:
             out = ops.diff_combine(out, self.diff.lam, self.diff.coef, self.diff.eps)
         return self.o(out.view(T, (self.heads // self.maps) * self.v_dim))
+
+    # ---- the layer's first product taken into a wider one (``parts.pair``) ----
+
+    def input_projections(self) -> Linear | None:
+        """The projection of ``x`` whose rows ``forward_projected`` takes, or None where ``x`` is read elsewhere too."""
+        return self.qkv if self.gate is None else None
+
+    def forward_projected(self, proj: torch.Tensor, ctx: StepContext, call: int) -> torch.Tensor:
+        """``forward`` from the rows of ``input_projections`` (a column block of wider rows)."""
+        out = self._heads(proj, None, ctx, call)
+        if self.diff is not None:
+            out = ops.diff_combine(out, self.diff.lam, self.diff.coef, self.diff.eps)
+        return self.o(out.view(proj.shape[0], (self.heads // self.maps) * self.v_dim))
 
     def _heads(self, proj: torch.Tensor, x: torch.Tensor | None, ctx: StepContext, call: int) -> torch.Tensor:
         """From the fused projection's rows to the gated heads' outputs [T, H, D]."""
@@ -253,6 +304,13 @@ class Attention:
             elif gate is not None:
                 ops.sigmoid_gate(out, gate)
             return out
+        if self.shape is not None:
+            out = self._attend_shaped(q, pool, table, ctx)
+            if gate is not None and self.gate_kind == "head":
+                ops.head_gate(out, gate, self.heads, self.v_dim)
+            elif gate is not None:
+                ops.sigmoid_gate(out, gate)
+            return out
         # the tensor-core kernels take everything but value heads of another size than the keys
         if self.v_dim == self.head_dim and ops.attention_mma_supported(self.heads, self.kv_heads, self.head_dim,
                                                                        q.dtype):
@@ -308,6 +366,37 @@ class Attention:
         return ops.attention_pointwise(q, pool, ctx.positions, ctx.tok_seq, table, tok0, ntok, per_tile, self.window,
                                        self.scale, self.v_dim, w.cap, w.temp_coef, w.temp_every, w.r1, w.r2,
                                        w.head_bias)
+
+    # whether capped and biased scores may take the tensor-core kernels (TOKENOMOS_B200_ATTN_BIASED_MMA=0: never)
+    biased_mma = os.environ.get("TOKENOMOS_B200_ATTN_BIASED_MMA", "1") != "0"
+
+    def _attend_shaped(self, q, pool, table, ctx: StepContext) -> torch.Tensor:
+        """Softmax attention with a cap and a distance bias on its scores: the tensor-core kernels where they take the
+        sizes (bfloat16), prompt portions in tiles of 64 rows and single tokens shared out over their keys; else the
+        general kernel."""
+        sh = self.shape
+        T = q.shape[0]
+        if self.biased_mma and ops.attention_biased_mma_supported(self.heads, self.kv_heads, self.head_dim, self.v_dim,
+                                                                  pool.shape[-1], q.dtype):
+            out = torch.empty(T, self.heads, self.v_dim, dtype=q.dtype, device=q.device)
+            tok0 = ntok = singles = None
+            n_single, nsplit = ctx.n_tokens, 1
+            if not ctx.host.decode_only:
+                _, tok0, _, ntok = ctx.tiles(ops.attention_biased_mma_tokens(self.heads, self.kv_heads), "multi")
+                singles = ctx.singles()
+                n_single = singles.numel()
+            if n_single:
+                longest = ctx.host.longest
+                if self.window is not None:
+                    longest = min(longest, self.window)
+                nsplit = self.decode_splits(n_single, self.kv_heads, longest, self.tuning)
+            ops.attention_biased_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, singles, n_single, nsplit,
+                                     self.window, self.scale, sh.cap, sh.bias, self.shape_bounded)
+            return out
+        per_tile = max(1, ops.attention_rows() // (self.heads // self.kv_heads))
+        _, tok0, _, ntok = ctx.tiles(per_tile)
+        return ops.attention(q, pool, ctx.positions, ctx.tok_seq, table, tok0, ntok, per_tile, self.window, self.scale,
+                             v_dim=self.v_dim, round_p=not self.exact, cap=sh.cap, bias=sh.bias)
 
     # whether prompt portions may take the tcgen05 kernel (TOKENOMOS_B200_ATTN_TC=0: never)
     prefill_tc = os.environ.get("TOKENOMOS_B200_ATTN_TC", "1") != "0"
@@ -413,6 +502,27 @@ def _diff(params: dict | None, tensors: dict) -> DiffMaps | None:
     return DiffMaps(lam, 1.0 - init, float(params["eps"]))
 
 
+def _shape(params: dict | None, tensors: dict, heads: int, window: int | None) -> ScoreShape | None:
+    """``params``: ``cap`` (absent or 0: none), ``bias_max`` (with the tensor ``rel`` [rows, heads]): the distance from
+    which on the last row of the table holds. The table is spread out by distance once, as far as the window or
+    ``bias_max`` reaches."""
+    if params is None:
+        return None
+    bias, rel = None, tensors.get("rel")
+    if rel is not None:
+        rows, far = rel.shape[0], float(params["bias_max"])
+        if far <= rows / 2:
+            raise ValueError(f"attention: a distance bias of {rows} rows up to a distance of {far:g}")
+        reach = max(int(math.ceil(far)), rows) + 1
+        if window is not None:
+            reach = max(1, min(reach, window))
+        index = torch.tensor([distance_bucket(n, rows, far) for n in range(reach)], device=rel.device)
+        bias = rel.float()[index].t().contiguous()
+        if bias.shape[0] != heads:
+            raise ValueError(f"attention: a distance bias for {bias.shape[0]} of {heads} heads")
+    return ScoreShape(float(params.get("cap") or 0.0), bias)
+
+
 @register("mixer", "attention")
 def build_attention(params: dict, tensors: dict, rt: Runtime) -> Attention:
     rope_spec = params["position"]
@@ -446,4 +556,5 @@ def build_attention(params: dict, tensors: dict, rt: Runtime) -> Attention:
         gate_fused=gated, tuning=rt.tuning, sink=params.get("sink", False),
         keep_first=params.get("keep_first", 0), v_dim=params.get("v_dim"), v_is_k=v_is_k,
         gate_kind=params.get("gate_kind", "head"), exact=params.get("exact", False),
-        pointwise=_pointwise(params.get("pointwise"), tensors), diff=_diff(params.get("diff"), tensors))
+        pointwise=_pointwise(params.get("pointwise"), tensors), diff=_diff(params.get("diff"), tensors),
+        shape=_shape(params.get("shape"), tensors, params["heads"], params.get("window")))

@@ -107,14 +107,45 @@ class ClampedGLU:
 
 @register("feed_forward", "glu_clamped")
 def build_clamped_glu(params: dict, tensors: dict, rt: Runtime) -> ClampedGLU:
+    gate_up, run = _fused_gate_up(tensors, rt)
+    return ClampedGLU(gate_up, Linear(tensors["down"], tensors.get("down_bias"), tuning=rt.tuning), params.get("limit"),
+                      params.get("alpha", 1.0), params.get("shift", 0.0), run=run)
+
+
+class GeluGLU:
+    """Gated feed-forward with the tanh form of gelu: ``down(gelu_tanh(gate(x)) * up(x))``; gate and up are one fused
+    projection (gate first), every projection may have a bias. ``run``: as ``ClampedGLU``'s."""
+
+    capture_safe = True
+
+    def __init__(self, gate_up: Linear, down: Linear, run: int = 0):
+        if gate_up.out_features != 2 * down.in_features:
+            raise ValueError("GeluGLU: gate_up must be twice as wide as down's input")
+        self.gate_up, self.down, self.run = gate_up, down, run
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        w = self.gate_up.weight
+        if self.run == RUN and x.shape[0] <= self.gate_up.tuning.swiglu_fused_rows and ops.gemm_skinny_ok(x, w):
+            self.gate_up.note("skinny+gelu")
+            act = ops.gemm_skinny_gelu(x, w, self.gate_up.bias)
+        else:
+            act = ops.glu_gelu(self.gate_up(x), self.run)
+        return self.down(act)
+
+
+def _fused_gate_up(tensors: dict, rt: Runtime) -> tuple[Linear, int]:
+    """Gate and up as one projection, and the run length in which their rows alternate."""
     gate, up = tensors["gate"], tensors["up"]
     biases = [tensors.get("gate_bias"), tensors.get("up_bias")]
-    down = Linear(tensors["down"], tensors.get("down_bias"), tuning=rt.tuning)
-    args = (params.get("limit"), params.get("alpha", 1.0), params.get("shift", 0.0))
     if gate.dtype == torch.bfloat16 and gate.shape[0] % RUN == 0:
         bias = None
         if biases[0] is not None:
             bias = interleave_rows(biases[0].float().view(-1, 1), biases[1].float().view(-1, 1), RUN).view(-1)
-        return ClampedGLU(Linear(interleave_rows(gate, up, RUN), bias, tuning=rt.tuning), down, *args, run=RUN)
-    gate_up = Linear.fused([gate, up], biases if biases[0] is not None else None, tuning=rt.tuning)
-    return ClampedGLU(gate_up, down, *args)
+        return Linear(interleave_rows(gate, up, RUN), bias, tuning=rt.tuning), RUN
+    return Linear.fused([gate, up], biases if biases[0] is not None else None, tuning=rt.tuning), 0
+
+
+@register("feed_forward", "glu_gelu")
+def build_gelu_glu(params: dict, tensors: dict, rt: Runtime) -> GeluGLU:
+    gate_up, run = _fused_gate_up(tensors, rt)
+    return GeluGLU(gate_up, Linear(tensors["down"], tensors.get("down_bias"), tuning=rt.tuning), run)

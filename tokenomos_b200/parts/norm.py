@@ -79,30 +79,40 @@ class StreamNorm32:
 
     ``groups`` > 1: the row is split into that many equal consecutive parts and each is divided by its
     own root mean square (the weight still covers the whole row). A ``GatedRows`` handed in as ``pre``
-    gates what is added: ``stream' = stream + x * sigmoid(gate)``."""
+    gates what is added: ``stream' = stream + x * sigmoid(gate)``. Another ``StreamNorm32`` handed in as ``pre``
+    norms what is added (a norm behind the sublayer): ``stream' = stream + mult * norm(x)`` with that norm's weight,
+    eps and ``mult``, the add and both norms in one kernel; ``mult`` belongs to a norm in that place only."""
 
     capture_safe = True
     stream_dtype = torch.float32
 
     def __init__(self, weight: torch.Tensor, eps: float, offset: float = 0.0,
-                 store: torch.dtype = torch.float32, groups: int = 1):
+                 store: torch.dtype = torch.float32, groups: int = 1, mult: float = 1.0):
         self.weight = (weight.float() + float(offset)).contiguous()
         self.eps = float(eps)
         self.width = weight.numel()
         self.store = store
         self.groups = int(groups)
+        self.mult = float(mult)
+        self.scaled = self.weight if self.mult == 1.0 else (self.weight * self.mult).contiguous()
         if self.groups < 1 or self.width % self.groups:
             raise ValueError(f"rmsnorm32: a row of {self.width} in {groups} groups")
 
     def add_norm(self, x: torch.Tensor, residual: torch.Tensor | None, pre=None, wide: bool = False):
         """``stream = residual + x (+ pre.rows)``; returns ``(norm(stream), stream)``. ``x`` alone may
         be the stream itself (float32 in a 16-bit model) or the rows that start one. ``pre``: a
-        ``PendingAdd`` or None (no post-norm can be taken into the add). ``wide``: the normed rows
+        ``PendingAdd``, a ``GatedRows``, the sublayer's own post-norm or None. ``wide``: the normed rows
         also unrounded: returns ``(norm(stream), the same in float32, stream)``."""
+        if self.mult != 1.0:
+            raise ValueError("rmsnorm32: a factor on the normed rows belongs to a norm behind a sublayer")
+        if isinstance(pre, StreamNorm32):
+            if wide or self.groups > 1 or pre.groups > 1:
+                raise ValueError("rmsnorm32: behind a sublayer's norm neither norms in groups nor unrounded rows are built")
+            return ops.stream32_post_norm(residual, x, pre.scaled, pre.eps, self.weight, self.eps)
         if self.groups > 1 or isinstance(pre, GatedRows):
             return self._in_groups(x, residual, pre, wide)
         if pre is not None and not isinstance(pre, PendingAdd):
-            raise ValueError("StreamNorm32: no post-norm can be taken into the add")
+            raise ValueError("StreamNorm32: only a rmsnorm32 can be the norm behind a sublayer")
         more = pre.rows if pre is not None else None
         if residual is None and x.dtype == torch.float32 and (self.store != torch.float32 or more is not None):
             return ops.stream32_add_norm(x, None, self.weight, self.eps, rows_add=more, out_dtype=self.store,
@@ -126,7 +136,7 @@ class StreamNorm32:
 @register("norm", "rmsnorm32")
 def build_stream_norm32(params: dict, tensors: dict, rt: Runtime) -> StreamNorm32:
     norm = StreamNorm32(tensors["weight"], params["eps"], params.get("offset", 0.0), rt.dtype,
-                        params.get("groups", 1))
+                        params.get("groups", 1), params.get("mult", 1.0))
     # taps of a convolution on what a sublayer behind this norm reads (``parts.parallel``): the
     # arrangement that has one finds them here
     norm.input_taps = tensors.get("taps")

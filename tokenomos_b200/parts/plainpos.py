@@ -7,9 +7,14 @@ go into the paged pool and the queries come back as the attention kernels take t
 reads part m of both. The part hands each map to the kernels as a head of its own, of the key's full
 width with zeros outside its part, so that the kernels' ``q . k`` is the map's score against keys that are
 stored once (``[T, heads, maps, dim] -> [T, heads * maps, maps * dim]``).
+
+``q_norm`` / ``k_norm``: an RMS norm over a token's whole query row and whole key row (all heads at once, before they
+are split) with weights of those sizes, in the same kernel as the write.
 """
 
 from __future__ import annotations
+
+import torch
 
 from tokenomos_b200 import ops
 from tokenomos_b200.parts.contract import HeadLayout, StepContext
@@ -19,20 +24,29 @@ from tokenomos_b200.parts.registry import Runtime, register
 class PlainQKV:
     capture_safe = True
 
-    def __init__(self, maps: int = 1):
+    def __init__(self, maps: int = 1, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
+                 eps: float = 0.0):
         self.maps = int(maps)
         if self.maps < 1:
             raise ValueError(f"plain q/k/v: {maps} maps")
+        if self.maps > 1 and q_norm is not None:
+            raise ValueError("plain q/k/v: norms over the whole rows go with one map a head")
+        self.q_norm = q_norm.float().reshape(-1).contiguous() if q_norm is not None else None
+        self.k_norm = k_norm.float().reshape(-1).contiguous() if k_norm is not None else None
+        self.eps = float(eps)
 
     def encode_qk(self, qkv, ctx: StepContext, heads: HeadLayout, pool, table):
         if heads.q_norm is not None or heads.k_norm is not None or heads.v_is_k:
             raise ValueError("plain q/k/v: per-head norms and values that are the keys are not built here")
         if heads.heads % self.maps or heads.head_dim % self.maps:
             raise ValueError(f"plain q/k/v: {heads.heads} heads of {heads.head_dim} in {self.maps} maps")
+        if self.q_norm is not None:
+            return ops.qkv_row_norm_write(qkv, self.q_norm, self.k_norm, self.eps, ctx.positions, ctx.tok_seq, table, pool,
+                                          heads.heads, heads.kv_heads, heads.head_dim, heads.v_dim or heads.head_dim)
         return ops.qkv_maps_write(qkv, ctx.positions, ctx.tok_seq, table, pool, heads.heads // self.maps,
                                   heads.kv_heads, heads.head_dim // self.maps, heads.v_dim or heads.head_dim, self.maps)
 
 
 @register("position", "plain")
 def build_plain_qkv(params: dict, tensors: dict, rt: Runtime) -> PlainQKV:
-    return PlainQKV(params.get("maps", 1))
+    return PlainQKV(params.get("maps", 1), tensors.get("q_norm"), tensors.get("k_norm"), params.get("eps", 0.0))

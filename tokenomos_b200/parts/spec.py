@@ -22,9 +22,20 @@ ROLE_IDENTITY = "identity"    # small square float32 table around the identity; 
 ROLES = (ROLE_MATRIX, ROLE_EMBEDDING, ROLE_NORM, ROLE_VECTOR, ROLE_TABLE, ROLE_IDENTITY)
 
 
+class FreeDim(int):
+    """A dimension that the configuration does not give: the stored tensors do. Its ``name`` ties it to every other
+    dimension of that name, which must be stored with the same size; its value is what the random-weights mode makes
+    it."""
+
+    def __new__(cls, name: str, default: int):
+        self = super().__new__(cls, default)
+        self.name = name
+        return self
+
+
 @dataclass(frozen=True)
 class TensorDecl:
-    """One tensor of the checkpoint: its name, the exact shape it must have, how it is kept."""
+    """One tensor of the checkpoint: its name, the exact shape it must have (but for ``FreeDim``s), how it is kept."""
 
     name: str
     shape: tuple[int, ...]

@@ -20,7 +20,7 @@ import torch
 from safetensors import safe_open
 
 from tokenomos_b200.parts.spec import (ROLE_EMBEDDING, ROLE_IDENTITY, ROLE_MATRIX, ROLE_NORM, ROLE_TABLE,
-                                       ROLE_VECTOR, TensorDecl)
+                                       ROLE_VECTOR, FreeDim, TensorDecl)
 
 
 class WeightError(ValueError):
@@ -75,7 +75,8 @@ class Checkpoint:
 
 def check(source, decls: list[TensorDecl], scope: tuple[str, ...] = ()) -> None:
     """Raise ``WeightError`` unless ``source`` (``names()``, ``shape(name)``) holds the declared
-    tensors (optional ones may be absent) with the declared shapes, and nothing undeclared
+    tensors (optional ones may be absent) with the declared shapes (a ``FreeDim`` is whatever is
+    stored, the same wherever its name appears), and nothing undeclared
     under the name prefixes in ``scope`` (empty: under any name)."""
     have = set(source.names())
     declared = {d.name: d for d in decls}
@@ -83,11 +84,16 @@ def check(source, decls: list[TensorDecl], scope: tuple[str, ...] = ()) -> None:
     unexpected = sorted(n for n in have - set(declared)
                         if not scope or any(n.startswith(prefix) for prefix in scope))
     wrong = []
+    free: dict[str, int] = {}      # sizes the stored tensors give (``FreeDim``), by name, as first met
     for n, d in declared.items():
         if n in have:
             got = tuple(source.shape(n))
-            if got != tuple(d.shape):
-                wrong.append(f"{n}: stored {list(got)}, the configuration needs {list(d.shape)}")
+            need = tuple(d.shape)
+            if len(got) == len(need):
+                need = tuple(free.setdefault(want.name, size) if isinstance(want, FreeDim) else want
+                             for want, size in zip(need, got))
+            if got != need:
+                wrong.append(f"{n}: stored {list(got)}, the configuration needs {list(map(int, need))}")
     if missing or unexpected or wrong:
         parts = []
         if missing:
