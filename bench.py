@@ -1786,6 +1786,256 @@ def fakelorn_kernels(z: dict, pk: dict) -> list[dict]:
     return rows
 
 
+# ---------------------------------------------------------------------------------------------
+# --design tifisun: the Tifisun decoder beside Fakelorn (the other design with a recurrent state per head behind a
+# short convolution, windowed softmax attention and a 32-bit stream) at equal sizes
+# ---------------------------------------------------------------------------------------------
+
+TIFISUN_SIZES = {
+    "width2048": dict(width=2048, layers=6, heads=16, kv_heads=8, dim=128, vdim=128, taps=4, att_heads=16, att_kv=4,
+                      att_dim=128, att_vdim=128, window=1024, mem_heads=16, mem_dim=128, mem_vdim=128, ff=6144, vocab=65536),
+    "width1024": dict(width=1024, layers=6, heads=16, kv_heads=8, dim=64, vdim=64, taps=4, att_heads=16, att_kv=4,
+                      att_dim=64, att_vdim=64, window=1024, mem_heads=16, mem_dim=64, mem_vdim=64, ff=4096, vocab=65536),
+}
+
+
+def tifisun_config(z: dict) -> dict:
+    """Groups of three layers: delta rule with a decay per head, attention and lightning attention side by side, delta
+    rule with a decay per key channel; dense feed-forwards."""
+    delta = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "conv": z["taps"]}
+    pair = {"left": {"heads": z["att_heads"], "kv_heads": z["att_kv"], "dim": z["att_dim"], "vdim": z["att_vdim"],
+                     "scale": z["att_dim"] ** -0.5, "softcap": 20.0, "bias_max": z["window"], "mask": {"size": z["window"]}},
+            "right": {"heads": z["mem_heads"], "dim": z["mem_dim"], "vdim": z["mem_vdim"],
+                      "decay": [1.0 - 2.0 ** (-3.0 - 0.5 * h) for h in range(z["mem_heads"])]}}
+    kinds = (("delta", delta), ("parallel", pair), ("channel_delta", dict(delta, kv_heads=z["heads"])))
+    layers = [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": {"kind": "dense", "ff": z["ff"]}}
+              for i in range(z["layers"])]
+    return {"architecture": "Tifisun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "embedding": {"scale": 3.0}, "layers": layers}
+
+
+def tifisun_like_config(z: dict) -> dict:
+    """Fakelorn at the same sizes: state-space layers of the same state where Tifisun has delta rules, differential
+    attention of the same heads, window and cache where it has the pair."""
+    dense = {"kind": "dense", "ff": z["ff"]}
+    ssm = {"type": "mamba2", "mixer": {"heads": z["heads"], "vdim": z["vdim"], "state": z["dim"], "groups": z["kv_heads"],
+                                       "conv": z["taps"], "norm_groups": z["heads"]}, "mlp": dense}
+    diff = {"type": "attention", "mixer": {"heads": z["att_heads"], "kv_heads": z["att_kv"], "dim": z["att_dim"] // 2,
+                                           "vdim": z["att_vdim"], "scale": (z["att_dim"] // 2) ** -0.5, "diff": 0.5,
+                                           "mask": {"size": z["window"]}}, "mlp": dense}
+    return {"architecture": "Fakelorn", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [diff if i % 3 == 1 else ssm for i in range(z["layers"])]}
+
+
+def tifisun_prefill_flops(z: dict, tokens: int) -> float:
+    """Multiply-adds times two of one prompt of ``tokens`` tokens as the design defines it (the recurrences as an update
+    and a read of their state per token, three passes for the delta rules)."""
+    W, H, K, D, V = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"]
+    windowed = sum(min(i + 1, z["window"]) for i in range(tokens))
+    flops = 0.0
+    for i in range(z["layers"]):
+        kind = i % 3
+        if kind == 1:
+            Ha, Ga, Da, Va = z["att_heads"], z["att_kv"], z["att_dim"], z["att_vdim"]
+            Hm, Dm, Vm = z["mem_heads"], z["mem_dim"], z["mem_vdim"]
+            per_tok = W * (Ha * Da + Ga * (Da + Va) + Ha * Va) + W * (2 * Hm * Dm + 3 * Hm * Vm) + 2 * Hm * Dm * Vm
+            flops += 2.0 * windowed * Ha * (Da + Va)
+        else:
+            k = K if kind == 0 else H
+            per_tok = W * (2 * k * D + 2 * H * V) + 3 * H * D * V
+            per_tok += W * (H * V + 2 * H) if kind == 0 else W * (D + V + H) + D * H * D + V * H * V
+        flops += 2.0 * tokens * (per_tok + 3 * W * z["ff"])
+    return flops + 2.0 * z["vocab"] * W
+
+
+def tifisun_like_flops(z: dict, tokens: int) -> float:
+    W, H, K, D, V = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"]
+    windowed = sum(min(i + 1, z["window"]) for i in range(tokens))
+    flops = 0.0
+    for i in range(z["layers"]):
+        if i % 3 == 1:
+            Ha, Ga, Da, Va = z["att_heads"], z["att_kv"], z["att_dim"], z["att_vdim"]
+            per_tok = W * (Ha * Da + Ga * (Da + Va) + Ha * Va)
+            flops += 2.0 * windowed * Ha * (Da + 2 * Va)
+        else:
+            per_tok = W * (3 * H * V + 2 * K * D + H) + 2 * H * D * V
+        flops += 2.0 * tokens * (per_tok + 2 * W * W + 3 * W * z["ff"])
+    return flops + 2.0 * z["vocab"] * W
+
+
+def tifisun_kernels(z: dict, pk: dict) -> list[dict]:
+    """Each kernel the Tifisun path adds beside the kernel of an earlier model that does the like work, on the shapes of a
+    2,048-token prompt portion of one sequence (or 64 decoded tokens behind 2,048 positions), L2 flushed before every
+    launch, CUDA events around one call, median of 20 (5 for the long ones). ``frac``: bytes over time against the
+    measured copy bandwidth, or flops over time against the measured bf16 rate."""
+    import torch
+
+    from tokenomos_b200 import ops
+    from tokenomos_b200.parts.attention import ScoreShape
+
+    bf, dev = torch.bfloat16, "cuda"
+    T, W, P = 2048, z["width"], 16
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    rows = []
+
+    def add(name, ours_us, theirs_us, ours_work, theirs_work, unit, like):
+        peak = pk["hbm_gbs"] * 1e3 if unit == "bytes" else pk["bf16_tflops"] * 1e6       # per microsecond
+        fo = ours_work / ours_us / peak
+        row = {"kernel": name, "like": like, "unit": unit, "tifisun_us": round(ours_us, 1), "tifisun_frac": round(fo, 4)}
+        if theirs_us is not None:
+            ft = theirs_work / theirs_us / peak
+            row.update(like_us=round(theirs_us, 1), like_frac=round(ft, 4), times_further_from_roofline=round(ft / fo, 2))
+        rows.append(row)
+
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    pos = torch.arange(T, dtype=torch.int32, device=dev)
+    seq = torch.zeros(T, dtype=torch.int32, device=dev)
+    cu, zero1, one1 = i32([0, T]), i32([0]), i32([1])
+
+    # 1. the stream: norm of what is added, add, norm; beside Fakelorn's gated add + norm
+    nw = torch.ones(W, device=dev)
+    res32 = torch.randn(T, W, device=dev)
+    y, gate = torch.randn(T, W, device=dev).to(bf), torch.randn(T, W, device=dev).to(bf)
+    add("post-norm + residual add + norm",
+        _timed_us(lambda: ops.stream32_post_norm(res32, y, nw, 1e-6, nw, 1e-6), flush),
+        _timed_us(lambda: ops.stream32_group_norm(res32, y, gate, nw, 1e-6, 4, bf), flush),
+        T * W * (4 + 2 + 4 + 2), T * W * (4 + 2 + 2 + 4 + 2), "bytes", "Fakelorn: gated residual add + norm")
+    add("pair of outputs: two norms, mean",
+        _timed_us(lambda: ops.pair_norm_mean(y, gate, nw, nw, 1e-6), flush),
+        _timed_us(lambda: ops.stream32_group_norm(res32, y, gate, nw, 1e-6, 4, bf), flush),
+        T * W * 6, T * W * (4 + 2 + 2 + 4 + 2), "bytes", "Fakelorn: gated residual add + norm")
+    gu = torch.randn(T, 2 * z["ff"], device=dev).to(bf)
+    add("gelu-gated activation", _timed_us(lambda: ops.glu_gelu(gu, 8), flush), _timed_us(lambda: ops.swiglu(gu, 8), flush),
+        T * z["ff"] * 6, T * z["ff"] * 6, "bytes", "Fakelorn: SwiGLU activation")
+
+    # 2. attention: row norms + cache write; prompt and decode attention with cap and bias
+    H, G, D, V, win = z["att_heads"], z["att_kv"], z["att_dim"], z["att_vdim"], z["window"]
+    pages = T // P + 1
+    pool = torch.zeros(pages, 2, G, P, max(D, V), dtype=bf, device=dev)
+    tbl = torch.arange(1, pages, dtype=torch.int32, device=dev).view(1, -1)
+    qkv = torch.randn(T, H * D + G * (D + V), device=dev).to(bf)
+    wq, wk = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev)
+    add("query and key row norms + cache write",
+        _timed_us(lambda: ops.qkv_row_norm_write(qkv, wq, wk, 1e-6, pos, seq, tbl, pool, H, G, D, V), flush),
+        _timed_us(lambda: ops.qkv_maps_write(qkv, pos, seq, tbl, pool, H, G, D // 2, V, 2), flush),
+        T * (H * D + G * (D + V)) * 4, T * ((H * D + G * (D + V)) * 2 + 2 * H * D * 2 + G * (D + V) * 2), "bytes",
+        "Fakelorn: queries as maps + cache write")
+    q = ops.qkv_row_norm_write(qkv, wq, wk, 1e-6, pos, seq, tbl, pool, H, G, D, V)
+    bias = torch.randn(H, win, device=dev) * 0.3
+    bounded = ScoreShape(20.0, bias).bounded
+    windowed = sum(min(i + 1, win) for i in range(T))
+    per = ops.attention_biased_mma_tokens(H, G)
+    t0 = torch.arange(0, T, per, dtype=torch.int32, device=dev)
+    nt = torch.full_like(t0, per)
+    out = torch.empty(T, H, V, dtype=bf, device=dev)
+    if D == V and ops.attention_mma_supported(H, G, D, bf):
+        tc = ops.attention_prefill_tc_supported(H, G, D, bf)
+        per1 = (ops.attention_prefill_tc_tokens if tc else ops.attention_prefill_mma_tokens)(H, G)
+        t01 = torch.arange(0, T, per1, dtype=torch.int32, device=dev)
+        nt1 = torch.full_like(t01, per1)
+        qd = ops.qkv_maps_write(qkv, pos, seq, tbl, pool, H, G, D // 2, V, 2)
+        outd = torch.empty_like(qd)
+        perd = (ops.attention_prefill_tc_tokens if tc else ops.attention_prefill_mma_tokens)(2 * H, G)
+        t0d = torch.arange(0, T, perd, dtype=torch.int32, device=dev)
+        ntd = torch.full_like(t0d, perd)
+
+        def ours():
+            ops.attention_biased_mma(q, pool, out, pos, seq, tbl, t0, nt, None, 0, 1, win, D ** -0.5, 20.0, bias, bounded)
+
+        def plain():
+            if tc:
+                ops.attention_prefill_tc(q, pool, out, pos, seq, tbl, t01, nt1, win, D ** -0.5, None, 1)
+            else:
+                ops.attention_prefill_mma(q, pool, out, pos, seq, tbl, t01, nt1, win, D ** -0.5)
+
+        def diff():
+            if tc:
+                ops.attention_prefill_tc(qd, pool, outd, pos, seq, tbl, t0d, ntd, win, D ** -0.5, None, 1)
+            else:
+                ops.attention_prefill_mma(qd, pool, outd, pos, seq, tbl, t0d, ntd, win, D ** -0.5)
+            return ops.diff_combine(outd, 0.3, 0.5, 1e-6)
+
+        kind = "tcgen05" if tc else "mma.sync"
+        ours_us = _timed_us(ours, flush, reps=5)
+        add("prompt attention, cap and distance bias (mma.sync)", ours_us, _timed_us(diff, flush, reps=5),
+            2.0 * windowed * H * (D + V), 2.0 * windowed * H * (D + 2 * V), "flops",
+            f"Fakelorn: differential prompt attention ({kind}) + join")
+        add("prompt attention, cap and distance bias (mma.sync)", ours_us, _timed_us(plain, flush, reps=5),
+            2.0 * windowed * H * (D + V), 2.0 * windowed * H * (D + V), "flops", f"plain softmax prompt attention ({kind})")
+        Bd = 64
+        dpos = torch.full((Bd,), T - 1, dtype=torch.int32, device=dev)
+        dseq = torch.arange(Bd, dtype=torch.int32, device=dev)
+        dtbl = tbl.expand(Bd, -1).contiguous()
+        dq, dqd = q[:Bd].contiguous(), qd[:Bd].contiguous()
+        dout, doutd = torch.empty(Bd, H, V, dtype=bf, device=dev), torch.empty_like(dqd)
+
+        def diff_decode():
+            ops.attention_decode_mma(dqd, pool, doutd, dpos, dseq, dtbl, None, win, D ** -0.5, 2)
+            return ops.diff_combine(doutd, 0.3, 0.5, 1e-6)
+
+        kv_bytes = Bd * G * min(T, win) * (D + V) * 2
+        ours_us = _timed_us(lambda: ops.attention_biased_mma(dq, pool, dout, dpos, dseq, dtbl, None, None, None, Bd, 2, win,
+                                                             D ** -0.5, 20.0, bias, bounded), flush)
+        add("decode attention, cap and distance bias, 64 tokens", ours_us, _timed_us(diff_decode, flush), kv_bytes, kv_bytes,
+            "bytes", "Fakelorn: differential decode attention + join")
+        add("decode attention, cap and distance bias, 64 tokens", ours_us,
+            _timed_us(lambda: ops.attention_decode_mma(dq, pool, dout, dpos, dseq, dtbl, None, win, D ** -0.5, 2), flush),
+            kv_bytes, kv_bytes, "bytes", "plain softmax decode attention")
+
+    # 3. the recurrences, beside the state-space scan at equal state size
+    Hs, K, N, Vs = z["heads"], z["kv_heads"], z["dim"], z["vdim"]
+    inner = Hs * Vs
+    cu64 = torch.arange(0, T + 1, T // 64, dtype=torch.int32, device=dev)
+    z64, o64 = torch.zeros(64, dtype=torch.int32, device=dev), torch.arange(1, 65, dtype=torch.int32, device=dev)
+    cu1 = torch.arange(0, 65, dtype=torch.int32, device=dev)
+
+    def scans(Hx, Kx, Nx, Vx):
+        u = torch.randn(T, 2 * Kx * Nx + Hx * Vx, device=dev).to(bf)
+        S = torch.zeros(66, Hx, Vx, Nx, device=dev)
+        zb = torch.randn(T, Hx, device=dev)
+        za = torch.randn(T, Hx * Nx, device=dev)
+        db, dbc, A = torch.zeros(Hx, device=dev), torch.zeros(Hx * Nx, device=dev), torch.ones(Hx, device=dev)
+        off = (0, Kx * Nx, 2 * Kx * Nx)
+
+        def run(rule, decay, cu_, ctx_, slot_, n, t=T):
+            if rule == "add":
+                return ops.linmem_scan(u[:t], off, "add", "fixed", A, S, cu_, ctx_, slot_, n, Hx, Kx, Nx, Vx, act=True)
+            return ops.linmem_scan(u[:t], off, "delta", decay, A, S, cu_, ctx_, slot_, n, Hx, Kx, Nx, Vx, Nx ** -0.5, unit=True,
+                                   beta=zb[:t], gates=(za if decay == "channel" else zb)[:t], bias=dbc if decay == "channel" else db)
+        return run
+
+    def ssm(Hx, Gx, Nx, Vx):
+        xbc = torch.randn(T, Hx * Vx + 2 * Gx * Nx, device=dev).to(bf) * 0.5
+        dt = torch.randn(T, Hx, device=dev)
+        zero, ones = torch.zeros(Hx, device=dev), torch.ones(Hx, device=dev)
+        S = torch.zeros(66, Hx, Nx, Vx, device=dev)
+        return lambda cu_, ctx_, slot_, n, t=T: ops.ssd_scan(xbc[:t], dt[:t], zero, zero, ones, S, cu_, ctx_, slot_, n, Hx, Vx, Nx, Gx)
+
+    cases = (("delta rule, decay per head", "delta", "head", (Hs, K, N, Vs)),
+             ("delta rule, decay per channel", "delta", "channel", (Hs, Hs, N, Vs)),
+             ("lightning attention", "add", "fixed", (z["mem_heads"], z["mem_heads"], z["mem_dim"], z["mem_vdim"])))
+    for name, rule, decay, (Hx, Kx, Nx, Vx) in cases:
+        run, like = scans(Hx, Kx, Nx, Vx), ssm(Hx, Kx, Nx, Vx)
+        passes = 3 if rule == "delta" else 2
+        ours_f, like_f = 2.0 * T * Hx * Nx * Vx * passes, 2.0 * T * Hx * Nx * Vx * 2
+        add(f"{name}: scan over 2,048 tokens of one sequence", _timed_us(lambda: run(rule, decay, cu, zero1, one1, 1), flush, reps=5),
+            _timed_us(lambda: like(cu, zero1, one1, 1), flush, reps=5), ours_f, like_f, "flops",
+            "Fakelorn: state-space scan at equal state size (both 32-bit; of the bf16 tensor rate)")
+        add(f"{name}: scan over 2,048 tokens of 64 sequences", _timed_us(lambda: run(rule, decay, cu64, z64, o64, 64), flush, reps=5),
+            _timed_us(lambda: like(cu64, z64, o64, 64), flush, reps=5), ours_f, like_f, "flops", "Fakelorn: state-space scan")
+        add(f"{name}: one token of 64 sequences", _timed_us(lambda: run(rule, decay, cu1, o64, o64, 64, 64), flush),
+            _timed_us(lambda: like(cu1, o64, o64, 64, 64), flush), 64 * Hx * Nx * Vx * 8, 64 * Hx * Nx * Vx * 8, "bytes",
+            "Fakelorn: state-space scan")
+    yv = torch.randn(T, inner, device=dev)
+    zg = torch.randn(T, inner, device=dev).to(bf)
+    gw = torch.ones(inner, device=dev)
+    for name, groups, kind in (("head norm + gate", Hs, "silu"), ("row norm + gate", 1, "sigmoid")):
+        add(name, _timed_us(lambda: ops.norm_gate(yv, zg, gw, 1e-6, groups, kind), flush),
+            _timed_us(lambda: ops.gated_group_norm(yv, zg, gw, 1e-6, groups), flush), T * inner * 8, T * inner * 8, "bytes",
+            "Fakelorn: gate + norm in groups")
+    return rows
+
+
 def run_design(name: str, args, warmup: int) -> int:
     """``--design darizen``: decode (batch 8 and 64) and prefill (2,048 tokens) throughput of
     Darizen stacks at a few real layer sizes, beside the LFM3 stack of sliding-window attention
@@ -1798,7 +2048,8 @@ def run_design(name: str, args, warmup: int) -> int:
     from tokenomos_b200.weights import write_model_folder
 
     pk = peaks()
-    sizes = {"laposun": LAPOSUN_SIZES, "lisorax": LISORAX_SIZES, "fakelorn": FAKELORN_SIZES}.get(name, DESIGN_SIZES)
+    sizes = {"laposun": LAPOSUN_SIZES, "lisorax": LISORAX_SIZES, "fakelorn": FAKELORN_SIZES,
+             "tifisun": TIFISUN_SIZES}.get(name, DESIGN_SIZES)
     for size, z in sizes.items():
         if getattr(args, "design_size", None) and size != args.design_size:
             continue
@@ -1810,6 +2061,8 @@ def run_design(name: str, args, warmup: int) -> int:
             arms = (("lisorax", lisorax_config(z)), ("laposun", laposun_config(z)))
         elif name == "fakelorn":
             arms = (("fakelorn", fakelorn_config(z)), ("laposun", laposun_config(z)))
+        elif name == "tifisun":
+            arms = (("tifisun", tifisun_config(z)), ("fakelorn", tifisun_like_config(z)))
         else:
             arms = (("darizen", darizen_config(z)), ("lfm3", lfm3_like_config(z)))
         for arm, config in arms:
@@ -1833,14 +2086,16 @@ def run_design(name: str, args, warmup: int) -> int:
                 res[f"decode_b{batch}"] = {"tok_s": round(d["tok_s"], 1), "ms_per_step": round(d["ms_per_step"], 4),
                                            "launches": d["launches_per_step"]}
             pf = device_prefill(model, cfg, args.page)
-            flops = {"laposun": laposun_prefill_flops, "lisorax": lisorax_prefill_flops, "fakelorn": fakelorn_prefill_flops}.get(
+            flops = {"laposun": laposun_prefill_flops, "lisorax": lisorax_prefill_flops, "tifisun": tifisun_prefill_flops,
+                     "fakelorn": tifisun_like_flops if name == "tifisun" else fakelorn_prefill_flops}.get(
                 arm, lambda *_: pf["flops"])(z, pf["tokens"])
             res["prefill_2048"] = {"tok_s": round(pf["tok_s"], 1), "ms": round(pf["ms"], 3),
                                    "frac": round(flops / (pf["ms"] * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)}
             line[arm] = res
             del model
             torch.cuda.empty_cache()
-        line["kernels"] = {"laposun": laposun_kernels, "lisorax": lisorax_kernels, "fakelorn": fakelorn_kernels}.get(
+        line["kernels"] = {"laposun": laposun_kernels, "lisorax": lisorax_kernels, "fakelorn": fakelorn_kernels,
+                           "tifisun": tifisun_kernels}.get(
             name, design_kernels)(z, pk)
         print(json.dumps(line), flush=True)
     return 0
@@ -1870,9 +2125,9 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points")
     ap.add_argument("--trace", default=None,
                     help="--workload: write one JSON record per step of an extra pass to this file")
-    ap.add_argument("--design", default=None, choices=["darizen", "laposun", "lisorax", "fakelorn"],
+    ap.add_argument("--design", default=None, choices=["darizen", "laposun", "lisorax", "fakelorn", "tifisun"],
                     help="the named design beside the closest existing model at equal sizes instead (darizen beside "
-                         "LFM3, laposun beside darizen, lisorax beside laposun, fakelorn beside laposun)")
+                         "LFM3, laposun beside darizen, lisorax beside laposun, fakelorn beside laposun, tifisun beside fakelorn)")
     ap.add_argument("--design-size", default=None, help="only this size of the design's table")
     ap.add_argument("--sweep", action="store_true",
                     help="decode and prefill at other batch sizes and context lengths instead")

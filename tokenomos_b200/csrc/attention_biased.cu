@@ -28,11 +28,15 @@ enum : int { TK_K_ATTN_BIASED = 14 };
 
 struct BiasedOptions {
     float scale, cap;
-    const float* bias;       // [H, L] or null
+    const float* bias;       // [H, L] times log2(e), or null
     int L, window, D, Dv, Dp;
 };
 
 
+
+__device__ __forceinline__ void cp_async4(uint32_t dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(dst), "l"(src));
+}
 
 // Copies of 64 rows of W columns (D of them real) out of pages with rows Dp apart, NT threads; the page numbers of
 // a tile are looked up while the tile before it is in flight.
@@ -83,7 +87,7 @@ struct BiasedRows {
     const float* bias[2];    // the staged bias at the tile's first key: bias[-key]
 };
 
-template <int DK, int DV, int NK, bool BOUNDED>
+template <int DK, int DV, int NK, bool BOUNDED, bool MASK>
 __device__ __forceinline__ void biased_block(const uint32_t (&qf)[DK / 16][4], uint32_t ktile, uint32_t vtile, int k0, int j0,
                                              const BiasedRows& rows, bool capped, float c1, float k2, int window,
                                              float (&m)[2], float (&l)[2], float (&o)[DV / 8][4]) {
@@ -112,7 +116,7 @@ __device__ __forceinline__ void biased_block(const uint32_t (&qf)[DK / 16][4], u
         for (int e = 0; e < 4; ++e) {
             const int key = k0 + n * 8 + 2 * t + (e & 1);
             const int dist = rows.pos[e >> 1] - (j0 + key);                  // a padding row's position is -1
-            const bool visible = dist >= 0 && (window <= 0 || dist < window);
+            const bool visible = !MASK || (dist >= 0 && (window <= 0 || dist < window));
             const float b = rows.bias[e >> 1][-key];
             const float v = capped ? fmaf(-k2, rcp_approx(1.f + fast_exp2(s[n][e] * c1)), b) : fmaf(s[n][e], c1, b);
             s[n][e] = visible ? v : -INFINITY;
@@ -196,7 +200,8 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
     extern __shared__ __align__(128) unsigned char smem_raw[];
     constexpr int K_BYTES = 64 * DK * 2, V_BYTES = 64 * DV * 2, STAGE = K_BYTES + V_BYTES;
     const uint32_t smem = (uint32_t)__cvta_generic_to_shared(smem_raw);      // [stage][K 64 x DK | V 64 x DV]
-    float* bias_s = reinterpret_cast<float*>(smem_raw + 2 * STAGE);          // [stage][G][span]
+    float* bias_s = reinterpret_cast<float*>(smem_raw + 2 * STAGE);          // [stage][G][span], base-2 logarithms
+    const uint32_t bias_at = smem + 2 * STAGE;
     const int G = H / Hkv;
     const int kvh = blockIdx.x % Hkv;
     // prompt tiles in reverse: a tile late in its sequence reads the most keys and starts first
@@ -221,6 +226,8 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
     const int lo = opt.window > 0 ? max(0, pos_first - opt.window + 1) : 0;
     const int j_begin = (lo / 64) * 64;
     const int row0 = SINGLE ? 0 : warp * 16;
+    if (opt.bias == nullptr)
+        for (int i = tid; i < 2 * G * span; i += 128) bias_s[i] = 0.f;
 
     uint32_t qf[DK / 16][4];
     biased_load_q<DK>(qf, q, row0, rows, tok0, G, H, kvh * G, opt.D);
@@ -271,15 +278,18 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
             for (int k = 0; k < PitchLoader<DK, 128>::PER; ++k) vl.page[k] = kl.page[k];
         }
         vl.issue(base + K_BYTES, pool, v_delta, j0, lo, pos_last);
+        // bias of the tile's distances: entry i is distance i + pos_first - (j0 + 63)
+        if (opt.bias != nullptr) {
+            const uint32_t bs = bias_at + (uint32_t)(b * G * span) * 4;
+            const int d0 = pos_first - j0 - 63;
+            for (int h = warp; h < G; h += 4) {
+                const float* src = opt.bias + (size_t)(kvh * G + h) * opt.L;
+                for (int i = lane; i < span; i += 32)
+                    cp_async4(bs + (uint32_t)(h * span + i) * 4, src + min(max(i + d0, 0), opt.L - 1));
+            }
+        }
         cp_async_commit();
         if (it + 1 < it1) lookup(it + 1);
-        // bias of the tile's distances: entry i is distance i + pos_first - (j0 + 63)
-        float* bs = bias_s + (size_t)b * G * span;
-        const int d0 = pos_first - j0 - 63;
-        for (int i = tid; i < G * span; i += 128) {
-            const int d = min(max(i % span + d0, 0), opt.L - 1);
-            bs[i] = opt.bias != nullptr ? LOG2E * opt.bias[(size_t)(kvh * G + i / span) * opt.L + d] : 0.f;
-        }
     };
     if (it0 < it1) {
         lookup(it0);
@@ -296,9 +306,13 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
         if (SINGLE) {
             const int k0 = warp * 16;
             if (w_pos_max >= j0 + k0 && (opt.window <= 0 || j0 + k0 + 15 > w_pos_min - opt.window))
-                biased_block<DK, DV, 16, BOUNDED>(qf, base, base + K_BYTES, k0, j0, br, capped, c1, k2, opt.window, m, l, o);
+                biased_block<DK, DV, 16, BOUNDED, true>(qf, base, base + K_BYTES, k0, j0, br, capped, c1, k2, opt.window, m, l, o);
         } else if (w_pos_max >= j0 && (opt.window <= 0 || j0 + 63 > w_pos_min - opt.window)) {
-            biased_block<DK, DV, 64, BOUNDED>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, opt.window, m, l, o);
+            // (every key of an inner tile is seen by every row of the warp, padding rows aside, which nothing reads)
+            if (j0 + 63 > w_pos_min || (opt.window > 0 && j0 <= w_pos_max - opt.window))
+                biased_block<DK, DV, 64, BOUNDED, true>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, opt.window, m, l, o);
+            else
+                biased_block<DK, DV, 64, BOUNDED, false>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, opt.window, m, l, o);
         }
     }
 #pragma unroll
@@ -423,7 +437,7 @@ TK_API int tk_attn_biased_mma_tokens(int H, int Hkv) { return 64 / (H / Hkv); }
 
 // Prompt portions: tiles of tk_attn_biased_mma_tokens tokens (first token and count per tile). Single tokens (`n_single`
 // > 0): the rows `singles` lists (null: rows 0 .. n_single - 1), each shared `nsplit` ways over its keys; part_o float32
-// [nsplit, n_single, H, Dv] and part_ml [nsplit, n_single, H, 2] when nsplit > 1. bias: float32 [H, L] or null; bounded:
+// [nsplit, n_single, H, Dv] and part_ml [nsplit, n_single, H, 2] when nsplit > 1. bias: float32 [H, L] times log2(e), or null; bounded:
 // 2 cap + the bias's reach, in base-2 logarithms, stays well inside a float's exponents.
 TK_API int tk_attn_biased_mma(const void* q, const void* kv_pool, void* out, const int* positions, const int* tok_seq,
                               const int* block_table, int bt_stride, const int* tile_tok0, const int* tile_ntok, int n_tiles,
@@ -491,7 +505,7 @@ __global__ void __launch_bounds__(256)
 qkv_row_norm_write_kernel(const T* qkv, int64_t stride, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
                           const int* positions, const int* tok_seq, const int* block_table, int bt_stride, T* q_out, T* pool,
                           int nq, int nk, int nv, int Hkv, int D, int Dv, int P, int Dp) {
-    __shared__ float red[33];
+    __shared__ float red[66];
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -504,9 +518,15 @@ qkv_row_norm_write_kernel(const T* qkv, int64_t stride, const float* __restrict_
 #pragma unroll
             for (int e = 0; e < VEC; ++e) ss = fmaf(to_f<T>(c.v[e]), to_f<T>(c.v[e]), ss);
         }
-        return block_sum(ss, red);
+        return ss;
     };
-    const float rq = 1.0f / sqrtf(squares(row, nq) / (float)nq + eps);
+    const T* k = row + nq;
+    const T* v = k + nk;
+    const bool write = pool != nullptr;
+    const int pos = positions[t];
+    const int page = write ? TK_PAGE(TK_K_ATTN_BIASED, block_table[(size_t)tok_seq[t] * bt_stride + pos / P]) : 0;
+    const float2 ss = block_sum2(make_float2(squares(row, nq), write ? squares(k, nk) : 0.f), red);
+    const float rq = 1.0f / sqrtf(ss.x / (float)nq + eps), rk = 1.0f / sqrtf(ss.y / (float)nk + eps);
     auto normed = [&](const T* x, int i, float rstd, const float* w) {
         Chunk c = *reinterpret_cast<const Chunk*>(x + i);
 #pragma unroll
@@ -515,12 +535,7 @@ qkv_row_norm_write_kernel(const T* qkv, int64_t stride, const float* __restrict_
     };
     for (int i = threadIdx.x * VEC; i < nq; i += blockDim.x * VEC)
         *reinterpret_cast<Chunk*>(q_out + (size_t)t * nq + i) = normed(row, i, rq, wq);
-    if (pool == nullptr) return;
-    const T* k = row + nq;
-    const T* v = k + nk;
-    const float rk = 1.0f / sqrtf(squares(k, nk) / (float)nk + eps);
-    const int pos = positions[t];
-    const int page = TK_PAGE(TK_K_ATTN_BIASED, block_table[(size_t)tok_seq[t] * bt_stride + pos / P]);
+    if (!write) return;
     // [page][K | V][head][slot in page][Dp]
     T* kd = pool + (((size_t)page * 2 + 0) * Hkv * P + pos % P) * Dp;
     T* vd = pool + (((size_t)page * 2 + 1) * Hkv * P + pos % P) * Dp;

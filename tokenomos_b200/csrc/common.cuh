@@ -123,6 +123,58 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     return red[32];
 }
 
+// Four neighbouring elements between memory and 32-bit registers (16-byte aligned, 8-byte for 16-bit storage).
+template <typename T>
+struct Quad {
+    static __device__ __forceinline__ float4 load(const T* p);
+    static __device__ __forceinline__ void store(T* p, float4 v);
+};
+template <>
+struct Quad<float> {
+    static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+    static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <>
+struct Quad<__nv_bfloat16> {
+    static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+        uint2 raw;
+        raw.x = *reinterpret_cast<const uint32_t*>(&a);
+        raw.y = *reinterpret_cast<const uint32_t*>(&b);
+        *reinterpret_cast<uint2*>(p) = raw;
+    }
+};
+
+// Two sums over a block at once; `red` holds 66 floats.
+__device__ __forceinline__ float2 block_sum2(float2 v, float* red) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int nwarp = (blockDim.x + 31) >> 5;
+    v.x = warp_sum(v.x);
+    v.y = warp_sum(v.y);
+    __syncthreads();  // `red` may still be read from an earlier call
+    if (lane == 0) {
+        red[2 * warp] = v.x;
+        red[2 * warp + 1] = v.y;
+    }
+    __syncthreads();
+    if (warp == 0) {
+        const float x = warp_sum(lane < nwarp ? red[2 * lane] : 0.f);
+        const float y = warp_sum(lane < nwarp ? red[2 * lane + 1] : 0.f);
+        if (lane == 0) {
+            red[64] = x;
+            red[65] = y;
+        }
+    }
+    __syncthreads();
+    return make_float2(red[64], red[65]);
+}
+
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 
 // ---- programmatic dependent launch -----------------------------------------------------------

@@ -23,10 +23,9 @@
 
 namespace {
 enum : int { TK_K_LINMEM = 13 };
-constexpr int LM_LANES = 8;      // lanes of a column
 constexpr int LM_COLS = 4;       // columns of a warp (times the columns per thread)
 constexpr int LM_TOK = 16;       // tokens of a stage
-constexpr int LM_PROD = 4;       // warps that stage the next tokens
+constexpr int LM_STAGES = 3;
 
 enum : int { LM_ADD = 0, LM_DELTA = 1 };
 enum : int { LM_FIXED = 0, LM_HEAD = 1, LM_CHANNEL = 2 };
@@ -37,9 +36,8 @@ struct LinMem {
     int q_off, k_off, v_off;
     const float* zb;             // [T, >= H] (delta)
     int64_t zb_stride;
-    const float* za;             // [T, >= H] or [T, >= H D]; the decay itself when `ready`
+    const float* za;             // [T, >= H] or [T, >= H D]
     int64_t za_stride;
-    int ready;
     const float* bias;           // [H] or [H D]
     const float* A;              // [H]: exp(A_log), or the fixed decays
     float* state;                // [slots, H, V, D]
@@ -198,111 +196,157 @@ __device__ __forceinline__ void lm_shape(const LinMem& m, int lane, float (&kv)[
     }
     if (lane == 0) *kq = s * mk * mq;
 }
-template <int DPL>
-__device__ __forceinline__ void lm_channel_decay(const LinMem& m, int row, int h, int lane, float A, float* gs) {
-#pragma unroll
-    for (int j = 0; j < DPL; ++j) {
-        const int d = lane + 32 * j;
-        float g = 1.f;
-        if (d < m.D) {
-            const float z = m.za[(size_t)row * m.za_stride + h * m.D + d];
-            g = m.ready ? z : lm_decay(z + m.bias[h * m.D + d], A);
-        }
-        gs[d] = g;
-    }
-}
 }  // namespace
 
-// Portions: a block owns 4 `cw` columns of a head of a sequence, a column per eight lanes of its first cw warps. The
-// last LM_PROD warps stage the next 16 tokens in shared memory while the others walk the 16 before.
-template <typename T, int R, int RULE, int DECAY>
-__global__ void __launch_bounds__(32 * (8 + LM_PROD))
-linmem_scan_kernel(const LinMem m, int cw) {
-    constexpr int DPL = R / 4, DP = 8 * R;               // the key size, padded
-    constexpr int VEC = DECAY == LM_CHANNEL ? 3 : 2;     // staged vectors per token
-    constexpr int PER = LM_TOK / LM_PROD;                // tokens a staging warp brings per stage
-    extern __shared__ __align__(16) float smem[];        // [2][k | q | a][TOK][DP], then [2][TOK][cols] values
-    __shared__ float kq_s[2][LM_TOK], beta_s[2][LM_TOK], a_s[2][LM_TOK];
+// Portions, first kernel: everything a token brings to the walk that does not depend on the state, formed once and laid
+// out as the walk reads it (32-bit, zeros past D and V): kq [K][T'][k | q][DP], decays [H][T'][DP] (per channel),
+// values [H][T'][VP], and per head and token (a, beta, k . q, -). T' = T + LM_TOK rows, so that a stage may read past the
+// last token. One block per token.
+struct LinMemPrep {
+    float *kq, *g, *v;
+    float4* sc;
+    int rows, VP;            // T', the values' padded size
+};
+
+template <typename T, int DPL, int RULE, int DECAY>
+__global__ void __launch_bounds__(256)
+linmem_prepare_kernel(const LinMem m, const LinMemPrep p) {
+    constexpr int DP = 32 * DPL;
+    extern __shared__ float kq_s[];                      // [K]
     pdl_launch_dependents();
     pdl_wait();
-    const int s = blockIdx.z, h = blockIdx.y, cols = LM_COLS * cw, c0 = blockIdx.x * cols;
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int kh = warp; kh < m.K; kh += 8) {
+        float kv[DPL], qv[DPL];
+        float* dst = p.kq + ((size_t)kh * p.rows + t) * 2 * DP;
+        lm_fetch<T, DPL>(m, t, kh * (m.H / m.K), lane, kv, qv);
+        lm_shape<DPL>(m, lane, kv, qv, dst, dst + DP, kq_s + kh);
+    }
+    const T* v = (const T*)m.qkv + (size_t)t * m.stride + m.v_off;
+    for (int i = threadIdx.x; i < m.H * p.VP; i += 256) {
+        const int h = i / p.VP, c = i % p.VP;
+        float x = c < m.V ? to_f<T>(v[h * m.V + c]) : 0.f;
+        p.v[((size_t)h * p.rows + t) * p.VP + c] = m.act ? lm_silu(x) : x;
+    }
+    if constexpr (DECAY == LM_CHANNEL) {
+        for (int i = threadIdx.x; i < m.H * DP; i += 256) {
+            const int h = i / DP, d = i % DP;
+            p.g[((size_t)h * p.rows + t) * DP + d] =
+                d < m.D ? lm_decay(m.za[(size_t)t * m.za_stride + h * m.D + d] + m.bias[h * m.D + d], m.A[h]) : 1.f;
+        }
+    }
+    __syncthreads();
+    for (int h = threadIdx.x; h < m.H; h += 256) {
+        float4 s = make_float4(m.A[h], 0.f, kq_s[h / (m.H / m.K)], 0.f);
+        if constexpr (RULE == LM_DELTA) s.y = 1.0f / (1.0f + expf(-m.zb[(size_t)t * m.zb_stride + h]));
+        if constexpr (DECAY == LM_HEAD) s.x = lm_decay(m.za[(size_t)t * m.za_stride + h] + m.bias[h], m.A[h]);
+        p.sc[(size_t)h * p.rows + t] = s;
+    }
+}
+
+__device__ __forceinline__ void lm_copy16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
+}
+
+// Portions, second kernel: a block owns LM_COLS * CPT columns a warp of a head of a sequence and walks the sequence's
+// tokens; stages of LM_TOK tokens are copied LM_STAGES - 1 ahead.
+template <int R, int RULE, int DECAY, int CPT>
+__global__ void __launch_bounds__(256)
+linmem_scan_kernel(const LinMem m, const LinMemPrep p) {
+    constexpr int DP = 8 * R;                            // the key size, padded
+    constexpr int VEC = DECAY == LM_CHANNEL ? 3 : 2;     // staged vectors per token
+    extern __shared__ __align__(16) float smem[];        // [stage][k | q per token, decays, values, scalars]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int s = blockIdx.z, h = blockIdx.y, cols = LM_COLS * CPT * warps, c0 = blockIdx.x * cols;
     const int first = m.cu_seqlens[s], len = m.cu_seqlens[s + 1] - first;
     if (len <= 0) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int r = lane & 7, col = c0 + warp * LM_COLS + (lane >> 3);
-    const bool walker = warp < cw;
-    const float A = m.A[h];
-    float* vs = smem + 2 * VEC * LM_TOK * DP;
-    float* st = m.state + (((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[s]) * m.H + h) * m.V + col) * m.D;
-    float2 S[R / 2];
-
-    auto stage = [&](int t0, int b) {                    // by the staging warps
-        const int pw = warp - cw;
-        float* ks = smem + (size_t)(b * VEC + 0) * LM_TOK * DP;
-        float* qs = smem + (size_t)(b * VEC + 1) * LM_TOK * DP;
-        float kv[PER][DPL], qv[PER][DPL];
-#pragma unroll
-        for (int i = 0; i < PER; ++i) {
-            const int t = min(t0 + pw + i * LM_PROD, len - 1);
-            lm_fetch<T, DPL>(m, first + t, h, lane, kv[i], qv[i]);
+    const int r = lane & 7, wc = warp * LM_COLS * CPT + (lane >> 3);        // this thread's first column of the block
+    const int stage_floats = LM_TOK * (VEC * DP + cols + 4);
+    const float* kq = p.kq + ((size_t)(h / (m.H / m.K)) * p.rows + first) * 2 * DP;
+    const float* g = DECAY == LM_CHANNEL ? p.g + ((size_t)h * p.rows + first) * DP : nullptr;
+    const float* v = p.v + ((size_t)h * p.rows + first) * p.VP + c0;
+    const float* sc = reinterpret_cast<const float*>(p.sc + (size_t)h * p.rows + first);
+    const int v_cols = min(cols, p.VP - c0);             // (VP and cols are whole 16-byte chunks)
+    auto issue = [&](int t0, int b) {
+        if (t0 < len) {
+            float* dst = smem + (size_t)b * stage_floats;
+            for (int i = threadIdx.x; i < LM_TOK * 2 * DP / 4; i += blockDim.x) lm_copy16(dst + 4 * i, kq + (size_t)t0 * 2 * DP + 4 * i);
+            dst += LM_TOK * 2 * DP;
+            if constexpr (DECAY == LM_CHANNEL) {
+                for (int i = threadIdx.x; i < LM_TOK * DP / 4; i += blockDim.x) lm_copy16(dst + 4 * i, g + (size_t)t0 * DP + 4 * i);
+                dst += LM_TOK * DP;
+            }
+            for (int i = threadIdx.x; i < LM_TOK * cols / 4; i += blockDim.x) {
+                const int t = i / (cols / 4), c = (i % (cols / 4)) * 4;
+                if (c < v_cols) lm_copy16(dst + t * cols + c, v + (size_t)(t0 + t) * p.VP + c);
+            }
+            dst += LM_TOK * cols;
+            for (int i = threadIdx.x; i < LM_TOK; i += blockDim.x) lm_copy16(dst + 4 * i, sc + 4 * (size_t)(t0 + i));
         }
-        // values of all tokens, a lane per column
-        for (int i = threadIdx.x - 32 * cw; i < LM_TOK * cols; i += 32 * LM_PROD) {
-            const int t = min(t0 + i / cols, len - 1), c = c0 + i % cols;
-            float v = c < m.V ? to_f<T>(((const T*)m.qkv)[(size_t)(first + t) * m.stride + m.v_off + h * m.V + c]) : 0.f;
-            vs[b * LM_TOK * cols + i] = m.act ? lm_silu(v) : v;
-        }
-        if (pw == 0 && lane < LM_TOK) {
-            const int row = first + min(t0 + lane, len - 1);
-            if constexpr (RULE == LM_DELTA) beta_s[b][lane] = 1.0f / (1.0f + expf(-m.zb[(size_t)row * m.zb_stride + h]));
-            if constexpr (DECAY == LM_HEAD) a_s[b][lane] = lm_decay(m.za[(size_t)row * m.za_stride + h] + m.bias[h], A);
-        }
-#pragma unroll
-        for (int i = 0; i < PER; ++i) {
-            const int tk = pw + i * LM_PROD;
-            lm_shape<DPL>(m, lane, kv[i], qv[i], ks + tk * DP, qs + tk * DP, &kq_s[b][tk]);
-            if constexpr (DECAY == LM_CHANNEL)
-                lm_channel_decay<DPL>(m, first + min(t0 + tk, len - 1), h, lane, A,
-                                      smem + (size_t)(b * VEC + 2) * LM_TOK * DP + tk * DP);
-        }
+        asm volatile("cp.async.commit_group;\n" ::);
     };
+#pragma unroll
+    for (int i = 0; i < LM_STAGES - 1; ++i) issue(i * LM_TOK, i);
 
-    if (walker) lm_load<R>(S, st, r, m.D, col < m.V && m.seq_ctx[s] > 0);
-    else stage(0, 0);
-    __syncthreads();
-    for (int t0 = 0, b = 0; t0 < len; t0 += LM_TOK, b ^= 1) {
-        if (walker) {
-            const int nt = min(LM_TOK, len - t0);
-            const float* ks = smem + (size_t)(b * VEC + 0) * LM_TOK * DP + 4 * r;
-            const float* qs = smem + (size_t)(b * VEC + 1) * LM_TOK * DP + 4 * r;
-            const float* gs = smem + (size_t)(b * VEC + VEC - 1) * LM_TOK * DP + 4 * r;
-            const float* vt = vs + b * LM_TOK * cols + warp * LM_COLS + (lane >> 3);
-            auto walk = [&](int t) {
-                return lm_step<R, RULE, DECAY>(S, ks + t * DP, qs + t * DP, gs + t * DP,
-                                               DECAY == LM_FIXED ? A : DECAY == LM_HEAD ? a_s[b][t] : 0.f, vt[t * cols],
-                                               RULE == LM_DELTA ? beta_s[b][t] : 0.f, kq_s[b][t]);
-            };
-            if (nt == LM_TOK) {
-                float keep = 0.f;
+    float* st = m.state + ((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[s]) * m.H + h) * m.V * m.D;
+    float2 S[CPT][R / 2];
+    const bool carried = m.seq_ctx[s] > 0;
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const int col = c0 + wc + LM_COLS * c;
+        lm_load<R>(S[c], st + (size_t)col * m.D, r, m.D, carried && col < m.V);
+    }
+    const int HV = m.H * m.V;
+    float* y = m.y + (size_t)first * HV + h * m.V + c0 + wc;
+    int b = 0;
+    for (int t0 = 0; t0 < len; t0 += LM_TOK) {
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(LM_STAGES - 2));
+        __syncthreads();                                 // the stage is there, and the one before it is read
+        issue(t0 + (LM_STAGES - 1) * LM_TOK, (b + LM_STAGES - 1) % LM_STAGES);
+        const float* base = smem + (size_t)b * stage_floats;
+        b = (b + 1) % LM_STAGES;
+        const float* ks = base + 4 * r;
+        const float* gs = base + LM_TOK * 2 * DP + 4 * r;
+        const float* vt = base + LM_TOK * VEC * DP + wc;
+        const float4* scs = reinterpret_cast<const float4*>(base + LM_TOK * (VEC * DP + cols));
+        auto walk = [&](int t, float (&o)[CPT]) {
+            const float4 c4 = scs[t];
+#pragma unroll
+            for (int c = 0; c < CPT; ++c)
+                o[c] = lm_step<R, RULE, DECAY>(S[c], ks + t * 2 * DP, ks + t * 2 * DP + DP, gs + t * DP, c4.x,
+                                               vt[t * cols + LM_COLS * c], c4.y, c4.z);
+        };
+        const int nt = min(LM_TOK, len - t0);
+        if (nt == LM_TOK) {
+            float keep[CPT];
 #pragma unroll 8
-                for (int t = 0; t < LM_TOK; ++t) {
-                    const float o = walk(t);
-                    if (r == (t & 7)) keep = o;
-                    if ((t & 7) == 7 && col < m.V)
-                        m.y[(size_t)(first + t0 + t - 7 + r) * m.H * m.V + h * m.V + col] = keep;
-                }
-            } else {
-                for (int t = 0; t < nt; ++t) {
-                    const float o = walk(t);
-                    if (r == 0 && col < m.V) m.y[(size_t)(first + t0 + t) * m.H * m.V + h * m.V + col] = o;
+            for (int t = 0; t < LM_TOK; ++t) {
+                float o[CPT];
+                walk(t, o);
+#pragma unroll
+                for (int c = 0; c < CPT; ++c) {
+                    if (r == (t & 7)) keep[c] = o[c];
+                    if ((t & 7) == 7 && c0 + wc + LM_COLS * c < m.V) y[(size_t)(t0 + t - 7 + r) * HV + LM_COLS * c] = keep[c];
                 }
             }
-        } else if (t0 + LM_TOK < len) {
-            stage(t0 + LM_TOK, b ^ 1);
+        } else {
+            for (int t = 0; t < nt; ++t) {
+                float o[CPT];
+                walk(t, o);
+#pragma unroll
+                for (int c = 0; c < CPT; ++c)
+                    if (r == 0 && c0 + wc + LM_COLS * c < m.V) y[(size_t)(t0 + t) * HV + LM_COLS * c] = o[c];
+            }
         }
-        __syncthreads();
     }
-    if (walker) lm_store<R>(S, st, r, m.D, col < m.V);
+    asm volatile("cp.async.wait_group 0;\n" ::);
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const int col = c0 + wc + LM_COLS * c;
+        lm_store<R>(S[c], st + (size_t)col * m.D, r, m.D, col < m.V);
+    }
 }
 
 // Steps of single tokens (a few a sequence at most): the state streams through, CPT columns a thread, so that many
@@ -349,10 +393,7 @@ linmem_token_kernel(const LinMem m) {
         if constexpr (DECAY == LM_CHANNEL) {
             for (int d = threadIdx.x; d < DP; d += blockDim.x) {
                 float g = 1.f;
-                if (d < m.D) {
-                    const float z = m.za[(size_t)row * m.za_stride + h * m.D + d];
-                    g = m.ready ? z : lm_decay(z + m.bias[h * m.D + d], A);
-                }
+                if (d < m.D) g = lm_decay(m.za[(size_t)row * m.za_stride + h * m.D + d] + m.bias[h * m.D + d], A);
                 gs[d] = g;
             }
         }
@@ -374,8 +415,8 @@ linmem_token_kernel(const LinMem m) {
 
 namespace {
 template <typename T, int R, int RULE, int DECAY>
-void lm_launch(const LinMem& m, int n_seqs, bool tokens, int sm_count, cudaStream_t stream) {
-    if (tokens) {
+void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_count, cudaStream_t stream) {
+    if (scratch == nullptr) {
         constexpr int CPT = R >= 32 ? 1 : 2;
         const int per_warp = LM_COLS * CPT;
         int warps = (m.V + per_warp - 1) / per_warp;
@@ -384,39 +425,61 @@ void lm_launch(const LinMem& m, int n_seqs, bool tokens, int sm_count, cudaStrea
         tk_launch(linmem_token_kernel<T, R, RULE, DECAY, CPT>, dim3(blocks, m.H, n_seqs), dim3(32 * warps), 0, stream, m);
         return;
     }
-    // as many columns a block as leave a block for every SM
-    int cw = 8;
-    while (cw > 2 && (m.V + LM_COLS * cw - 1) / (LM_COLS * cw) * m.H * n_seqs < sm_count) cw /= 2;
-    const int cols = LM_COLS * cw;
-    const size_t smem = (2 * (size_t)(DECAY == LM_CHANNEL ? 3 : 2) * LM_TOK * 8 * R + 2 * (size_t)LM_TOK * cols) * sizeof(float);
-    static size_t raised = 48 * 1024;
-    if (smem > raised) {
-        cudaFuncSetAttribute(linmem_scan_kernel<T, R, RULE, DECAY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        raised = smem;
+    constexpr int DP = 8 * R, VEC = DECAY == LM_CHANNEL ? 3 : 2;
+    LinMemPrep p;
+    p.rows = tokens + LM_TOK;
+    p.VP = (m.V + 3) / 4 * 4;
+    p.kq = scratch;
+    p.v = p.kq + (size_t)m.K * p.rows * 2 * DP;
+    p.sc = reinterpret_cast<float4*>(p.v + (size_t)m.H * p.rows * p.VP);
+    p.g = reinterpret_cast<float*>(p.sc + (size_t)m.H * p.rows);
+    tk_launch(linmem_prepare_kernel<T, R / 4, RULE, DECAY>, dim3(tokens), dim3(256), m.K * sizeof(float), stream, m, p);
+    auto scan = [&](auto kernel, int cpt, int warps) {
+        const int cols = LM_COLS * cpt * warps;
+        const size_t smem = (size_t)LM_STAGES * LM_TOK * (VEC * DP + cols + 4) * sizeof(float);
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        tk_launch(kernel, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * warps), smem, stream, m, p);
+    };
+    // few, long portions: a column a thread, as many columns a block as leave a block for every SM; else two
+    auto blocks = [&](int cols) { return (m.V + cols - 1) / cols * m.H * n_seqs; };
+    int warps = 8;
+    if (R < 32 && blocks(LM_COLS * 2 * 8) >= 2 * sm_count) {
+        while (warps > 2 && m.V <= LM_COLS * 2 * warps / 2) warps /= 2;
+        if constexpr (R < 32) scan(linmem_scan_kernel<R, RULE, DECAY, 2>, 2, warps);
+    } else {
+        while (warps > 2 && (blocks(LM_COLS * warps) < sm_count || m.V <= LM_COLS * warps / 2)) warps /= 2;
+        scan(linmem_scan_kernel<R, RULE, DECAY, 1>, 1, warps);
     }
-    tk_launch(linmem_scan_kernel<T, R, RULE, DECAY>, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * (cw + LM_PROD)),
-              smem, stream, m, cw);
 }
 
 template <typename T, int RULE, int DECAY>
-void lm_rows(const LinMem& m, int n_seqs, bool tokens, int sm_count, cudaStream_t stream) {
-    if (m.D <= 32) lm_launch<T, 4, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
-    else if (m.D <= 64) lm_launch<T, 8, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
-    else if (m.D <= 128) lm_launch<T, 16, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
-    else lm_launch<T, 32, RULE, DECAY>(m, n_seqs, tokens, sm_count, stream);
+void lm_rows(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_count, cudaStream_t stream) {
+    if (m.D <= 32) lm_launch<T, 4, RULE, DECAY>(m, n_seqs, tokens, scratch, sm_count, stream);
+    else if (m.D <= 64) lm_launch<T, 8, RULE, DECAY>(m, n_seqs, tokens, scratch, sm_count, stream);
+    else if (m.D <= 128) lm_launch<T, 16, RULE, DECAY>(m, n_seqs, tokens, scratch, sm_count, stream);
+    else lm_launch<T, 32, RULE, DECAY>(m, n_seqs, tokens, scratch, sm_count, stream);
 }
 }  // namespace
 
 TK_API int tk_linmem_max_dim() { return 256; }
 
+// Scratch memory of a step, in units of 32 floats: none for single tokens (a few a sequence at most), else what the
+// walk's vectors take.
+TK_API int tk_linmem_scratch(int tokens, int n_seqs, int H, int K, int D, int V, int decay) {
+    if (tokens < 4 * n_seqs || n_seqs == 0) return 0;
+    const int64_t DP = D <= 32 ? 32 : D <= 64 ? 64 : D <= 128 ? 128 : 256, VP = (V + 3) / 4 * 4;
+    const int64_t floats = (int64_t)(tokens + LM_TOK) * (2 * K * DP + H * (VP + 4) + (decay == LM_CHANNEL ? H * DP : 0));
+    return (int)((floats + 31) / 32);
+}
+
 // qkv: [T, >= ...] rows `stride` apart holding q (K x D) at column q_off, k at k_off, v (H x V) at v_off; rule 0
 // additive, 1 delta (zb: float32 [T, >= H] rows zb_stride apart, beta's logits); decay 0 fixed (A: float32 [H], the
 // decays), 1 per head, 2 per channel (za: float32 [T, >= H] or [T, >= H D] rows za_stride apart, bias likewise one
-// row, A: float32 [H]); ready: za holds the decays themselves. state: float32 [slots, H, V, D]; y: float32 [T, H V].
+// row, A: float32 [H]). scratch: what tk_linmem_scratch says (16-byte aligned), null for 0. state: float32 [slots, H, V, D]; y: float32 [T, H V].
 TK_API int tk_linmem_scan(const void* qkv, int64_t stride, int q_off, int k_off, int v_off, int rule, const float* zb,
-                          int64_t zb_stride, int decay, const float* za, int64_t za_stride, int ready, const float* bias,
+                          int64_t zb_stride, int decay, const float* za, int64_t za_stride, const float* bias,
                           const float* A, float* state, const int* cu_seqlens, const int* seq_ctx, const int* seq_slot,
-                          int n_seqs, int tokens, float* y, int H, int K, int D, int V, float q_scale, int unit, int act,
+                          int n_seqs, int tokens, float* y, float* scratch, int H, int K, int D, int V, float q_scale, int unit, int act,
                           int sm_count, int dtype, cudaStream_t stream) {
     TK_CHECK_ARG(H > 0 && K > 0 && H % K == 0 && D > 0 && V > 0, "linear memory: %d heads over %d q/k heads", H, K);
     TK_CHECK_ARG(D <= tk_linmem_max_dim(), "linear memory: a key size of %d; up to %d are built", D, tk_linmem_max_dim());
@@ -425,14 +488,15 @@ TK_API int tk_linmem_scan(const void* qkv, int64_t stride, int q_off, int k_off,
     TK_CHECK_ARG(rule == LM_ADD || (zb != nullptr && za != nullptr && bias != nullptr), "linear memory: missing gates");
     TK_CHECK_ARG(n_seqs >= 0 && tokens >= 0 && A != nullptr, "linear memory: bad sizes");
     if (n_seqs == 0) return 0;
-    const LinMem m{qkv, stride, q_off, k_off, v_off, zb, zb_stride, za, za_stride, ready, bias, A, state, cu_seqlens, seq_ctx,
+    const LinMem m{qkv, stride, q_off, k_off, v_off, zb, zb_stride, za, za_stride, bias, A, state, cu_seqlens, seq_ctx,
                    seq_slot, y, H, K, D, V, q_scale, unit, act};
-    const bool few = tokens < 4 * n_seqs;      // single tokens, not portions
+    TK_CHECK_ARG((scratch != nullptr) == (tk_linmem_scratch(tokens, n_seqs, H, K, D, V, decay) > 0),
+                 "linear memory: a step of %d tokens in %d sequences without its scratch memory", tokens, n_seqs);
 #define TK_LM(TT)                                                                       \
     do {                                                                                \
-        if (rule == LM_ADD) lm_rows<TT, LM_ADD, LM_FIXED>(m, n_seqs, few, sm_count, stream);          \
-        else if (decay == LM_HEAD) lm_rows<TT, LM_DELTA, LM_HEAD>(m, n_seqs, few, sm_count, stream);  \
-        else lm_rows<TT, LM_DELTA, LM_CHANNEL>(m, n_seqs, few, sm_count, stream);                     \
+        if (rule == LM_ADD) lm_rows<TT, LM_ADD, LM_FIXED>(m, n_seqs, tokens, scratch, sm_count, stream);          \
+        else if (decay == LM_HEAD) lm_rows<TT, LM_DELTA, LM_HEAD>(m, n_seqs, tokens, scratch, sm_count, stream);  \
+        else lm_rows<TT, LM_DELTA, LM_CHANNEL>(m, n_seqs, tokens, scratch, sm_count, stream);                     \
     } while (0)
     if (dtype == TK_F32) TK_LM(float);
     else if (dtype == TK_BF16) TK_LM(__nv_bfloat16);
@@ -526,40 +590,62 @@ TK_API int tk_norm_gate(const float* y, const void* z, int64_t z_stride, const f
 // Two mixers' outputs joined: out = coef * (a / rms(a) * wa + b / rms(b) * wb), rms over the row with
 // eps inside the root, in 32-bit with one rounding. One block per row.
 // ---------------------------------------------------------------------------------------------
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 pair_norm_mean_kernel(const T* a, int64_t a_stride, const T* b, int64_t b_stride, const float* __restrict__ wa,
                       const float* __restrict__ wb, float eps, float coef, T* out, int width) {
-    constexpr int ITEMS = 8;
-    __shared__ float red[33];
+    constexpr int ITEMS = 2;                              // steps of four elements that stay in registers
+    __shared__ float red[66];
     pdl_launch_dependents();
     pdl_wait();
     const size_t r = blockIdx.x;
     const T* pa = a + r * a_stride;
     const T* pb = b + r * b_stride;
-    float va[ITEMS], vb[ITEMS], sa = 0.f, sb = 0.f;
+    float2 ss = make_float2(0.f, 0.f);
+    if constexpr (VEC) {
+        auto square = [](float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+        float4 va[ITEMS], vb[ITEMS];
 #pragma unroll
-    for (int k = 0; k < ITEMS; ++k) {
-        const int i = threadIdx.x + k * blockDim.x;
-        va[k] = i < width ? to_f<T>(pa[i]) : 0.f;
-        vb[k] = i < width ? to_f<T>(pb[i]) : 0.f;
-        sa = fmaf(va[k], va[k], sa);
-        sb = fmaf(vb[k], vb[k], sb);
-    }
-    for (int i = threadIdx.x + ITEMS * blockDim.x; i < width; i += blockDim.x) {
-        const float x = to_f<T>(pa[i]), y = to_f<T>(pb[i]);
-        sa = fmaf(x, x, sa);
-        sb = fmaf(y, y, sb);
-    }
-    const float ra = coef / sqrtf(block_sum(sa, red) / (float)width + eps);
-    const float rb = coef / sqrtf(block_sum(sb, red) / (float)width + eps);
+        for (int k = 0; k < ITEMS; ++k) {
+            const int i = (threadIdx.x + k * blockDim.x) * 4;
+            va[k] = i < width ? Quad<T>::load(pa + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            vb[k] = i < width ? Quad<T>::load(pb + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
 #pragma unroll
-    for (int k = 0; k < ITEMS; ++k) {
-        const int i = threadIdx.x + k * blockDim.x;
-        if (i < width) out[r * width + i] = from_f<T>(va[k] * ra * wa[i] + vb[k] * rb * wb[i]);
+        for (int k = 0; k < ITEMS; ++k) {
+            ss.x += square(va[k]);
+            ss.y += square(vb[k]);
+        }
+        for (int i = (threadIdx.x + ITEMS * blockDim.x) * 4; i < width; i += blockDim.x * 4) {
+            ss.x += square(Quad<T>::load(pa + i));
+            ss.y += square(Quad<T>::load(pb + i));
+        }
+        ss = block_sum2(ss, red);
+        const float ra = coef / sqrtf(ss.x / (float)width + eps), rb = coef / sqrtf(ss.y / (float)width + eps);
+        auto join = [&](float4 x, float4 y, int i) {
+            const float4 p = *reinterpret_cast<const float4*>(wa + i), q = *reinterpret_cast<const float4*>(wb + i);
+            Quad<T>::store(out + r * width + i,
+                           make_float4(x.x * ra * p.x + y.x * rb * q.x, x.y * ra * p.y + y.y * rb * q.y,
+                                       x.z * ra * p.z + y.z * rb * q.z, x.w * ra * p.w + y.w * rb * q.w));
+        };
+#pragma unroll
+        for (int k = 0; k < ITEMS; ++k) {
+            const int i = (threadIdx.x + k * blockDim.x) * 4;
+            if (i < width) join(va[k], vb[k], i);
+        }
+        for (int i = (threadIdx.x + ITEMS * blockDim.x) * 4; i < width; i += blockDim.x * 4)
+            join(Quad<T>::load(pa + i), Quad<T>::load(pb + i), i);
+    } else {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            const float x = to_f<T>(pa[i]), y = to_f<T>(pb[i]);
+            ss.x = fmaf(x, x, ss.x);
+            ss.y = fmaf(y, y, ss.y);
+        }
+        ss = block_sum2(ss, red);
+        const float ra = coef / sqrtf(ss.x / (float)width + eps), rb = coef / sqrtf(ss.y / (float)width + eps);
+        for (int i = threadIdx.x; i < width; i += blockDim.x)
+            out[r * width + i] = from_f<T>(to_f<T>(pa[i]) * ra * wa[i] + to_f<T>(pb[i]) * rb * wb[i]);
     }
-    for (int i = threadIdx.x + ITEMS * blockDim.x; i < width; i += blockDim.x)
-        out[r * width + i] = from_f<T>(to_f<T>(pa[i]) * ra * wa[i] + to_f<T>(pb[i]) * rb * wb[i]);
 }
 
 // a, b: [rows, width] (type dtype) rows `a_stride` / `b_stride` apart; wa, wb: float32 [width]; out: [rows, width].
@@ -568,15 +654,21 @@ TK_API int tk_pair_norm_mean(const void* a, int64_t a_stride, const void* b, int
                              cudaStream_t stream) {
     TK_CHECK_ARG(rows >= 0 && width > 0, "pair_norm_mean: bad sizes rows=%d width=%d", rows, width);
     if (rows == 0) return 0;
-    const int threads = width >= 1024 ? 256 : 128;
-    if (dtype == TK_F32)
-        tk_launch(pair_norm_mean_kernel<float>, dim3(rows), dim3(threads), 0, stream, (const float*)a, a_stride,
-                  (const float*)b, b_stride, wa, wb, eps, coef, (float*)out, width);
-    else if (dtype == TK_BF16)
-        tk_launch(pair_norm_mean_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, (const __nv_bfloat16*)a,
-                  a_stride, (const __nv_bfloat16*)b, b_stride, wa, wb, eps, coef, (__nv_bfloat16*)out, width);
-    else
+    const int threads = width >= 1024 ? 256 : 128, es = dtype == TK_BF16 ? 2 : 4;
+    const bool vec = width % 4 == 0 && a_stride % 4 == 0 && b_stride % 4 == 0 && (((uintptr_t)wa | (uintptr_t)wb) & 15) == 0 &&
+                     (((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & (4 * es - 1)) == 0;
+#define TK_PM(TT, VEC)                                                                                              \
+    tk_launch(pair_norm_mean_kernel<TT, VEC>, dim3(rows), dim3(threads), 0, stream, (const TT*)a, a_stride, (const TT*)b, \
+              b_stride, wa, wb, eps, coef, (TT*)out, width)
+    if (dtype == TK_F32) {
+        if (vec) TK_PM(float, true);
+        else TK_PM(float, false);
+    } else if (dtype == TK_BF16) {
+        if (vec) TK_PM(__nv_bfloat16, true);
+        else TK_PM(__nv_bfloat16, false);
+    } else
         TK_CHECK_ARG(false, "pair_norm_mean: unknown dtype %d", dtype);
+#undef TK_PM
     TK_CHECK_LAUNCH("pair_norm_mean");
     return 0;
 }

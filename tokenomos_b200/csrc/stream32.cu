@@ -68,33 +68,6 @@ stream32_add_norm_kernel(const float* stream_in, const T* x, int64_t x_stride, c
 // The same with 16 bytes of the stream (four elements) per thread and step, the row in registers:
 // one trip to memory. Needs width % 4 == 0, rows of x a multiple of four elements apart, every
 // base 16-byte aligned (8-byte for 16-bit inputs), and width <= 4 * ITEMS * blockDim.
-template <typename T>
-struct Quad {
-    static __device__ __forceinline__ float4 load(const T* p);
-    static __device__ __forceinline__ void store(T* p, float4 v);
-};
-template <>
-struct Quad<float> {
-    static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
-    static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-};
-template <>
-struct Quad<__nv_bfloat16> {
-    static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
-        const uint2 raw = *reinterpret_cast<const uint2*>(p);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-        return make_float4(a.x, a.y, b.x, b.y);
-    }
-    static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
-        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-        uint2 raw;
-        raw.x = *reinterpret_cast<const uint32_t*>(&a);
-        raw.y = *reinterpret_cast<const uint32_t*>(&b);
-        *reinterpret_cast<uint2*>(p) = raw;
-    }
-};
-
 template <typename T, int ITEMS>
 __global__ void __launch_bounds__(256)
 stream32_add_norm_vec_kernel(const float* stream_in, const T* x, int64_t x_stride, const T* rows_add,

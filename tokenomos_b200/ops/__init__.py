@@ -1567,12 +1567,12 @@ def linmem_scan(qkv: torch.Tensor, offsets: tuple, rule: str, decay: str, A: tor
                 cu_seqlens: torch.Tensor, seq_ctx: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, heads: int, kv_heads: int,
                 dim: int, v_dim: int, q_scale: float = 1.0, unit: bool = False, act: bool = False,
                 beta: torch.Tensor | None = None, gates: torch.Tensor | None = None, bias: torch.Tensor | None = None,
-                ready: bool = False, sm_count: int = 148) -> torch.Tensor:
+                sm_count: int = 148) -> torch.Tensor:
     """A matrix memory per head over a step's tokens: ``S <- a S``, then ``S <- S + k v^T`` (``rule`` "add") or ``u =
     sigmoid(beta) (v - S^T k), S <- S + k u^T`` ("delta"), ``y = S^T q``. ``qkv`` [T, *]: q (``kv_heads`` x dim) at column
     ``offsets[0]``, k at ``offsets[1]``, v (``heads`` x v_dim) at ``offsets[2]``; head h reads q/k head ``h / (heads /
     kv_heads)``. ``decay``: "fixed" (``A`` float32 [heads] holds a), "head" or "channel" (``a = exp(-A[h] softplus(gates
-    + bias))`` with ``gates`` float32 [T, >= heads] or [T, >= heads dim]; ``ready``: ``gates`` holds a). ``act``: q, k
+    + bias))`` with ``gates`` float32 [T, >= heads] or [T, >= heads dim]). ``act``: q, k
     and v pass silu first; ``unit``: q and k are brought to unit length; q is multiplied by ``q_scale``. ``state`` float32
     [slots, heads, v_dim, dim]. Returns ``y`` float32 [T, heads v_dim]."""
     _cuda(qkv, A, state, beta, gates, bias)
@@ -1586,12 +1586,15 @@ def linmem_scan(qkv: torch.Tensor, offsets: tuple, rule: str, decay: str, A: tor
         if need and (t is None or t.dtype != torch.float32 or t.stride(1) != 1 or t.shape[0] != T or t.shape[1] < need):
             raise KernelError(f"linmem_scan: {name} is float32 [{T}, >= {need}] with contiguous columns")
     y = torch.empty(T, heads * v_dim, dtype=torch.float32, device=qkv.device)
+    # a step with portions stages its vectors in memory first
+    n = _lib.call("tk_linmem_scratch", T, int(n_seqs), heads, kv_heads, dim, v_dim, LINMEM_DECAYS[decay])
+    scratch = torch.empty(n, 32, dtype=torch.float32, device=qkv.device) if n else None
     _lib.call("tk_linmem_scan", _ptr(qkv), qkv.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]), LINMEM_RULES[rule],
               _ptr(beta), beta.stride(0) if beta is not None else 0, LINMEM_DECAYS[decay], _ptr(gates),
-              gates.stride(0) if gates is not None else 0, int(bool(ready)), _ptr(_f32vec(bias, "decay bias", cols)) if cols else None,
+              gates.stride(0) if gates is not None else 0, _ptr(_f32vec(bias, "decay bias", cols)) if cols else None,
               _ptr(_f32vec(A, "A", heads)), _ptr(state), _ptr(_i32(cu_seqlens, "cu_seqlens")), _ptr(_i32(seq_ctx, "seq_ctx")),
-              _ptr(_i32(seq_slot, "seq_slot")), int(n_seqs), T, _ptr(y), heads, kv_heads, dim, v_dim, float(q_scale),
-              int(bool(unit)), int(bool(act)), int(sm_count), _dtype_code(qkv), _stream())
+              _ptr(_i32(seq_slot, "seq_slot")), int(n_seqs), T, _ptr(y), _ptr(scratch), heads, kv_heads, dim, v_dim,
+              float(q_scale), int(bool(unit)), int(bool(act)), int(sm_count), _dtype_code(qkv), _stream())
     return y
 
 
@@ -1663,14 +1666,15 @@ def attention_biased_mma_tokens(heads: int, kv_heads: int) -> int:
 def attention_biased_mma(q: torch.Tensor, kv_pool: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,
                          tok_seq: torch.Tensor, block_table: torch.Tensor, tile_tok0: torch.Tensor | None,
                          tile_ntok: torch.Tensor | None, singles: torch.Tensor | None, n_single: int, nsplit: int,
-                         window: int | None, scale: float, cap: float = 0.0, bias: torch.Tensor | None = None,
+                         window: int | None, scale: float, cap: float = 0.0, bias_log2: torch.Tensor | None = None,
                          bounded: bool = False) -> None:
-    """Softmax attention with scores ``cap tanh(q.k scale / cap) + bias[h, min(i - j, L - 1)]`` on the tensor cores: the
+    """Softmax attention with scores ``cap tanh(q.k scale / cap) + bias[h, min(i - j, L - 1)]`` on the tensor cores
+    (``bias_log2`` is ``bias`` over ``ln 2``): the
     tiles of prompt portions (``attention_biased_mma_tokens`` tokens each) and ``n_single`` single tokens (their rows
     in ``singles``; None: rows 0 .. n_single - 1), each shared ``nsplit`` ways over its keys. ``q`` [T, H, D], ``out``
     [T, H, Dv], ``kv_pool`` [pages, 2, Hkv, P, row]. ``bounded``: cap and bias keep every score, in base-2 logarithms,
     well inside a float's exponents, so the softmax needs no running maximum."""
-    _cuda(q, kv_pool, out, positions, tok_seq, block_table, tile_tok0, tile_ntok, singles, bias)
+    _cuda(q, kv_pool, out, positions, tok_seq, block_table, tile_tok0, tile_ntok, singles, bias_log2)
     T, H, D = q.shape
     _, two, Hkv, P, Dp = kv_pool.shape
     Dv = out.shape[2]
@@ -1686,5 +1690,5 @@ def attention_biased_mma(q: torch.Tensor, kv_pool: torch.Tensor, out: torch.Tens
               _ptr(_i32(tok_seq, "tok_seq")), _ptr(_i32(block_table, "block_table")), block_table.stride(0),
               _ptr(_i32(tile_tok0, "tile_tok0")) if n_tiles else None, _ptr(_i32(tile_ntok, "tile_ntok")) if n_tiles else None,
               n_tiles, _ptr(_i32(singles, "singles")) if singles is not None else None, int(n_single), int(nsplit), _ptr(part_o),
-              _ptr(part_ml), H, Hkv, D, Dv, Dp, P, int(window or 0), float(scale), float(cap or 0.0), *_bias_table(bias, H),
+              _ptr(part_ml), H, Hkv, D, Dv, Dp, P, int(window or 0), float(scale), float(cap or 0.0), *_bias_table(bias_log2, H),
               int(bool(bounded)), _stream())

@@ -110,7 +110,8 @@ _SIGNATURES = {
     "tk_glu_gelu": [P, P, I, I, I, I, P],
     "tk_gemm_skinny_gelu": [P, L, P, L, P, P, L, I, I, I, I, P],
     "tk_linmem_max_dim": [],
-    "tk_linmem_scan": [P, L, I, I, I, I, P, L, I, P, L, I, P, P, P, P, P, P, I, I, P, I, I, I, I, F, I, I, I, I, P],
+    "tk_linmem_scratch": [I, I, I, I, I, I, I],
+    "tk_linmem_scan": [P, L, I, I, I, I, P, L, I, P, L, P, P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, I, I, I, P],
     "tk_norm_gate": [P, P, L, P, F, P, I, I, I, I, I, P],
     "tk_pair_norm_mean": [P, L, P, L, P, P, F, F, P, I, I, I, P],
     "tk_attn_biased_mma_supported": [I, I, I, I, I],
@@ -168,7 +169,7 @@ _QUERIES = {"tk_check_device", "tk_built_for", "tk_set_pdl", "tk_checks_enabled"
             "tk_attn_prefill_tc_tokens", "tk_attn_prefill_tc_status", "tk_gemm_tc_status", "tk_sample_status",
             "tk_attn_latent_rows", "tk_attn_latent_max_rank", "tk_gemm_grouped_tile", "tk_attn_latent_mma_rows",
             "tk_attn_latent_mma_supported", "tk_attn_pointwise_rows", "tk_attn_pointwise_mma_supported",
-            "tk_attn_pointwise_mma_tokens", "tk_ssd_max_state", "tk_ssd_split", "tk_linmem_max_dim",
+            "tk_attn_pointwise_mma_tokens", "tk_ssd_max_state", "tk_ssd_split", "tk_linmem_max_dim", "tk_linmem_scratch",
             "tk_attn_biased_mma_supported", "tk_attn_biased_mma_tokens"}
 
 

@@ -131,6 +131,8 @@ class Attention:
             if shape.bias is not None and shape.bias.shape[0] != heads:
                 raise ValueError(f"attention: a distance bias of {shape.bias.shape[0]} rows for {heads} heads")
             self.shape_bounded = shape.bounded          # (asked once: it reads the bias from the device)
+            # the tensor-core kernels carry scores in base-2 logarithms
+            self.bias_log2 = (shape.bias.double() / math.log(2.0)).float() if shape.bias is not None else None
         if pointwise is not None and (sink or keep_first):
             raise ValueError("attention: a sink and kept first positions belong to the softmax")
         # what the one-kernel decode form and the norms folded into the projections do not take
@@ -391,7 +393,7 @@ class Attention:
                     longest = min(longest, self.window)
                 nsplit = self.decode_splits(n_single, self.kv_heads, longest, self.tuning)
             ops.attention_biased_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, singles, n_single, nsplit,
-                                     self.window, self.scale, sh.cap, sh.bias, self.shape_bounded)
+                                     self.window, self.scale, sh.cap, self.bias_log2, self.shape_bounded)
             return out
         per_tile = max(1, ops.attention_rows() // (self.heads // self.kv_heads))
         _, tok0, _, ntok = ctx.tiles(per_tile)
