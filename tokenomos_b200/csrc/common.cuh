@@ -211,3 +211,16 @@ static inline cudaError_t tk_launch(void (*kernel)(KArgs...), dim3 grid, dim3 bl
     cfg.numAttrs = tk_pdl_enabled() ? 1 : 0;
     return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
+
+// A launch in plain stream order: for a long kernel of few blocks, whose blocks would otherwise be placed around
+// those of the kernel before it (several on one SM, none on another) and stay there for its whole run.
+template <typename... KArgs, typename... Args>
+static inline cudaError_t tk_launch_after(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                                          cudaStream_t stream, Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = stream;
+    return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+}

@@ -434,22 +434,21 @@ void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_c
     p.sc = reinterpret_cast<float4*>(p.v + (size_t)m.H * p.rows * p.VP);
     p.g = reinterpret_cast<float*>(p.sc + (size_t)m.H * p.rows);
     tk_launch(linmem_prepare_kernel<T, R / 4, RULE, DECAY>, dim3(tokens), dim3(256), m.K * sizeof(float), stream, m, p);
-    auto scan = [&](auto kernel, int cpt, int warps) {
-        const int cols = LM_COLS * cpt * warps;
-        const size_t smem = (size_t)LM_STAGES * LM_TOK * (VEC * DP + cols + 4) * sizeof(float);
-        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        tk_launch(kernel, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * warps), smem, stream, m, p);
-    };
-    // few, long portions: a column a thread, as many columns a block as leave a block for every SM; else two
-    auto blocks = [&](int cols) { return (m.V + cols - 1) / cols * m.H * n_seqs; };
-    int warps = 8;
-    if (R < 32 && blocks(LM_COLS * 2 * 8) >= 2 * sm_count) {
-        while (warps > 2 && m.V <= LM_COLS * 2 * warps / 2) warps /= 2;
-        if constexpr (R < 32) scan(linmem_scan_kernel<R, RULE, DECAY, 2>, 2, warps);
-    } else {
-        while (warps > 2 && (blocks(LM_COLS * warps) < sm_count || m.V <= LM_COLS * warps / 2)) warps /= 2;
-        scan(linmem_scan_kernel<R, RULE, DECAY, 1>, 1, warps);
+    // Two columns a thread (one where a column alone is 32 registers) in blocks of four warps; eight warps, which share
+    // a stage's copies among more columns, only where even a quarter of the sequences (the least a recorded step of
+    // this shape was recorded for) would fill the GPU with them
+    constexpr int CPT = R >= 32 ? 1 : 2;
+    int warps = (m.V + LM_COLS * CPT * 8 - 1) / (LM_COLS * CPT * 8) * m.H * (n_seqs / 4) >= sm_count ? 8 : 4;
+    while (warps > 1 && m.V <= LM_COLS * CPT * warps / 2) warps /= 2;
+    const int cols = LM_COLS * CPT * warps;
+    const size_t smem = (size_t)LM_STAGES * LM_TOK * (VEC * DP + cols + 4) * sizeof(float);
+    static size_t raised = 48 * 1024;
+    if (smem > raised) {
+        cudaFuncSetAttribute(linmem_scan_kernel<R, RULE, DECAY, CPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        raised = smem;
     }
+    tk_launch_after(linmem_scan_kernel<R, RULE, DECAY, CPT>, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * warps), smem,
+                    stream, m, p);
 }
 
 template <typename T, int RULE, int DECAY>
