@@ -3,7 +3,7 @@ per-request state of fixed size.
 
 What the model asks for arrives as ``StateSpec``s keyed by (entry of the layer list, name).
 Paged specs are sorted into *groups* by what they keep (every position, or a window of the last
-``w``); each group has its own pool of page numbers and its own block table per request, and
+``w``, or a chunk at a time); each group has its own pool of page numbers and its own block table per request, and
 every layer of the group indexes its own tensor ``[pages, 2, kv_heads, page, head_dim]`` with
 the group's page numbers. Pages return to the group's pool when the request ends, or, in a
 window group, as soon as no later query can see them (the pages of a group's kept first
@@ -76,6 +76,7 @@ class Group:
     pages: FreeList
     members: list[StateKey] = field(default_factory=list)
     keep_first: int = 0          # first positions of a sequence that a window never passes
+    chunk: int = 0               # positions are read chunk by chunk (``window`` is a chunk's size)
 
 
 @dataclass
@@ -125,10 +126,11 @@ class CacheManager:
             if storage == "paged":
                 g = self.groups.get(spec.group)
                 keep = int(getattr(spec, "keep_first", 0) or 0)
+                chunk = int(getattr(spec, "chunk", 0) or 0)
                 if g is None:
                     g = self.groups[spec.group] = Group(spec.group, spec.window, FreeList(num_pages),
-                                                        keep_first=keep)
-                elif g.window != spec.window or g.keep_first != keep:
+                                                        keep_first=keep, chunk=chunk)
+                elif g.window != spec.window or g.keep_first != keep or g.chunk != chunk:
                     raise ValueError(f"state {key}: cache group {spec.group} holds a window of "
                                      f"{g.window}, this spec asks for {spec.window}")
                 g.members.append(key)
@@ -215,7 +217,8 @@ class CacheManager:
         """First block a query at position ``ctx`` or later can read in group ``g``."""
         if g.window is None:
             return 0
-        return max(0, ctx - g.window + 1) // self.page_size
+        first = ctx - ctx % g.chunk if g.chunk else max(0, ctx - g.window + 1)
+        return first // self.page_size
 
     def pages_needed(self, rid, n_new: int) -> dict[tuple, int]:
         """Pages each group must still hand out so ``rid`` can take ``n_new`` more tokens."""

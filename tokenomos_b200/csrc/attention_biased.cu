@@ -1,9 +1,10 @@
 // Paged softmax attention with a soft cap on the scores and a learned bias by distance, on the tensor cores
 // (bfloat16, warp-level mma.sync m16n8k16):
 //
-//     s_ij = cap tanh((q_i . k_j) scale / cap) + bias[h][min(i - j, L - 1)],   softmax over 0 <= i - j < window
+//     s_ij = cap tanh((q_i . k_j) scale / cap) + bias[h][min(i - j, L - 1)],   softmax over first_seen(i, window) <= j <= i
 //
-// (cap 0: none; window <= 0: every earlier position). Keys and values may differ in size (D and Dv up to 128,
+// (cap 0: none; a sliding window, chunks or every earlier position: see first_seen). With a sink the softmax's denominator
+// has one more term, a key of score 0 without a value. Keys and values may differ in size (D and Dv up to 128,
 // multiples of 8; the cache row Dp holds either); the tiles in shared memory are 64 or 128 wide, columns past D
 // or Dv are zeros. Scores, bias, maxima and sums are 32-bit; a weight is rounded to bfloat16 where it meets the
 // values. The CUDA-core form for any sizes and 32-bit storage is attn_generic's.
@@ -14,8 +15,9 @@
 // The bias of a tile's distances (at most 63 + the tile's tokens of them) is staged beside its keys, per head.
 // With the cap as tanh(z) = 1 - 2 / (1 + e^(2 z)), a score in base-2 logarithms and up to a constant of the row is
 //     s2 = bias log2(e) - k2 / (1 + 2^(c1 dot)),    c1 = 2 scale log2(e) / cap,  k2 = 2 cap log2(e),
-// which lies between -k2 and 0 around the bias: where that range is narrow enough for 32-bit powers of two
-// (BOUNDED, decided by the caller from cap and bias) no running maximum is needed and shares simply add up.
+// which lies between -k2 and 0 around the bias (a sink, of score 0, is at -k2 / 2 there): where that range is narrow
+// enough for 32-bit powers of two (BOUNDED, decided by the caller from cap and bias, or, without a cap, from the lengths
+// of queries and keys) no running maximum is needed and shares simply add up.
 //
 // In front of it: the write of the step's keys and values with a norm over a token's whole query row and whole key
 // row (not per head), for layers whose positions enter through the scores alone.
@@ -29,7 +31,7 @@ enum : int { TK_K_ATTN_BIASED = 14 };
 struct BiasedOptions {
     float scale, cap;
     const float* bias;       // [H, L] times log2(e), or null
-    int L, window, D, Dv, Dp;
+    int L, window, D, Dv, Dp, sink;
 };
 
 
@@ -84,12 +86,13 @@ struct PitchLoader {
 // Rows of a warp: the two a lane works for (g and g + 8)
 struct BiasedRows {
     int pos[2];              // positions, -1: padding
+    int first[2];            // the first positions they see
     const float* bias[2];    // the staged bias at the tile's first key: bias[-key]
 };
 
 template <int DK, int DV, int NK, bool BOUNDED, bool MASK>
 __device__ __forceinline__ void biased_block(const uint32_t (&qf)[DK / 16][4], uint32_t ktile, uint32_t vtile, int k0, int j0,
-                                             const BiasedRows& rows, bool capped, float c1, float k2, int window,
+                                             const BiasedRows& rows, bool capped, float c1, float k2,
                                              float (&m)[2], float (&l)[2], float (&o)[DV / 8][4]) {
     const int lane = threadIdx.x & 31;
     const int t = lane & 3, mi = lane >> 3, r = lane & 7;
@@ -115,8 +118,8 @@ __device__ __forceinline__ void biased_block(const uint32_t (&qf)[DK / 16][4], u
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int key = k0 + n * 8 + 2 * t + (e & 1);
-            const int dist = rows.pos[e >> 1] - (j0 + key);                  // a padding row's position is -1
-            const bool visible = !MASK || (dist >= 0 && (window <= 0 || dist < window));
+            // (a padding row's position is -1)
+            const bool visible = !MASK || (j0 + key <= rows.pos[e >> 1] && j0 + key >= rows.first[e >> 1]);
             const float b = rows.bias[e >> 1][-key];
             const float v = capped ? fmaf(-k2, rcp_approx(1.f + fast_exp2(s[n][e] * c1)), b) : fmaf(s[n][e], c1, b);
             s[n][e] = visible ? v : -INFINITY;
@@ -223,7 +226,7 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
     const int g = lane >> 2;
     const int pos_first = positions[tok0];
     const int pos_last = pos_first + ntok - 1;       // consecutive positions within a tile
-    const int lo = opt.window > 0 ? max(0, pos_first - opt.window + 1) : 0;
+    const int lo = first_seen(pos_first, opt.window);
     const int j_begin = (lo / 64) * 64;
     const int row0 = SINGLE ? 0 : warp * 16;
     if (opt.bias == nullptr)
@@ -238,6 +241,7 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
         const int r = row0 + g + 8 * e;
         const bool ok = r < rows;
         br.pos[e] = ok ? pos_first + r / G : -1;
+        br.first[e] = first_seen(br.pos[e], opt.window);
         bias_off[e] = (ok ? (r % G) * span + r / G : 0) + 63;
     }
     const bool capped = opt.cap > 0.f;
@@ -247,8 +251,14 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
     const int w_last_row = min(rows, row0 + 16) - 1;
     const int w_pos_max = w_last_row >= row0 ? pos_first + w_last_row / G : -1;
     const int w_pos_min = pos_first + row0 / G;
+    const int w_first_min = first_seen(w_pos_min, opt.window), w_first_max = first_seen(w_pos_max, opt.window);
 
     float m[2] = {BOUNDED ? 0.f : -INFINITY, BOUNDED ? 0.f : -INFINITY}, l[2] = {0.f, 0.f};
+    if (opt.sink && (!SINGLE || (warp == 0 && blockIdx.y == 0))) {        // the sink joins a row's sum once
+        const float at = capped ? -0.5f * k2 : 0.f;
+        if constexpr (!BOUNDED) m[0] = m[1] = at;
+        if ((lane & 3) == 0) l[0] = l[1] = BOUNDED ? fast_exp2(at) : 1.f;
+    }
     float o[DV / 8][4];
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n)
@@ -305,14 +315,14 @@ attn_biased_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
         br.bias[1] = bias_s + (size_t)b * G * span + bias_off[1];
         if (SINGLE) {
             const int k0 = warp * 16;
-            if (w_pos_max >= j0 + k0 && (opt.window <= 0 || j0 + k0 + 15 > w_pos_min - opt.window))
-                biased_block<DK, DV, 16, BOUNDED, true>(qf, base, base + K_BYTES, k0, j0, br, capped, c1, k2, opt.window, m, l, o);
-        } else if (w_pos_max >= j0 && (opt.window <= 0 || j0 + 63 > w_pos_min - opt.window)) {
+            if (w_pos_max >= j0 + k0 && j0 + k0 + 15 >= w_first_min)
+                biased_block<DK, DV, 16, BOUNDED, true>(qf, base, base + K_BYTES, k0, j0, br, capped, c1, k2, m, l, o);
+        } else if (w_pos_max >= j0 && j0 + 63 >= w_first_min) {
             // (every key of an inner tile is seen by every row of the warp, padding rows aside, which nothing reads)
-            if (j0 + 63 > w_pos_min || (opt.window > 0 && j0 <= w_pos_max - opt.window))
-                biased_block<DK, DV, 64, BOUNDED, true>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, opt.window, m, l, o);
+            if (j0 + 63 > w_pos_min || j0 < w_first_max)
+                biased_block<DK, DV, 64, BOUNDED, true>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, m, l, o);
             else
-                biased_block<DK, DV, 64, BOUNDED, false>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, opt.window, m, l, o);
+                biased_block<DK, DV, 64, BOUNDED, false>(qf, base, base + K_BYTES, 0, j0, br, capped, c1, k2, m, l, o);
         }
     }
 #pragma unroll
@@ -438,19 +448,18 @@ TK_API int tk_attn_biased_mma_tokens(int H, int Hkv) { return 64 / (H / Hkv); }
 // Prompt portions: tiles of tk_attn_biased_mma_tokens tokens (first token and count per tile). Single tokens (`n_single`
 // > 0): the rows `singles` lists (null: rows 0 .. n_single - 1), each shared `nsplit` ways over its keys; part_o float32
 // [nsplit, n_single, H, Dv] and part_ml [nsplit, n_single, H, 2] when nsplit > 1. bias: float32 [H, L] times log2(e), or null; bounded:
-// 2 cap + the bias's reach, in base-2 logarithms, stays well inside a float's exponents.
+// the scores' reach, in base-2 logarithms, stays well inside a float's exponents. window: see first_seen.
 TK_API int tk_attn_biased_mma(const void* q, const void* kv_pool, void* out, const int* positions, const int* tok_seq,
                               const int* block_table, int bt_stride, const int* tile_tok0, const int* tile_ntok, int n_tiles,
                               const int* singles, int n_single, int nsplit, float* part_o, float* part_ml, int H, int Hkv,
                               int D, int Dv, int Dp, int P, int window, float scale, float cap, const float* bias, int L,
-                              int bounded, cudaStream_t stream) {
+                              int bounded, int sink, cudaStream_t stream) {
     TK_CHECK_ARG(tk_attn_biased_mma_supported(H, Hkv, D, Dv, Dp),
                  "attention: %d / %d heads of %d and %d are not the tensor-core form's", H, Hkv, D, Dv);
     TK_CHECK_ARG(P > 0 && n_tiles >= 0 && n_single >= 0 && cap >= 0.f && nsplit >= 1, "attention: bad sizes");
     TK_CHECK_ARG(nsplit == 1 || (part_o != nullptr && part_ml != nullptr), "attention: shares need scratch memory");
     TK_CHECK_ARG(bias == nullptr || L > 0, "attention: a distance bias of %d columns", L);
-    TK_CHECK_ARG(!bounded || cap > 0.f, "attention: scores without a cap have no bound");
-    const BiasedOptions opt{scale, cap, bias, max(L, 1), window, D, Dv, Dp};
+    const BiasedOptions opt{scale, cap, bias, max(L, 1), window, D, Dv, Dp, sink};
     const int G = H / Hkv, shift = biased_shift(P);
     auto q16 = (const __nv_bfloat16*)q;
     auto pool = (const __nv_bfloat16*)kv_pool;

@@ -5,8 +5,8 @@
 // included (the q/k kernel wrote them first). This is the path of the 32-bit model and the
 // fallback of the 16-bit one.
 //
-// Score s = (q.k) * scale, key j visible to a query at position i iff j <= i and (no window or
-// i - j < window or j < keep_first); online softmax; P rounded to the storage type before P.V
+// Score s = (q.k) * scale, key j visible to a query at position i iff j <= i and (j >= first_seen(i, window) or
+// j < keep_first); online softmax; P rounded to the storage type before P.V
 // when `round_p` (the 16-bit reference's rounding), else kept in 32-bit; the row sum keeps the
 // unrounded values (Tokenomos kernels/attention/paged.py:67-76,150,267;
 // models/blocks/attention.py:31-40,173).
@@ -72,11 +72,11 @@ attn_generic_kernel(const T* q, const T* kv_pool, T* out,
 
     const int pos_first = row_pos[0];
     const int pos_last = row_pos[rows - 1];
-    const int lo = window > 0 ? max(0, pos_first - window + 1) : 0;
+    const int lo = first_seen(pos_first, window);
 
     const int r = tid >> 3;   // my row
     const int sub = tid & 7;  // my lane within the row
-    const int my_pos = row_pos[r];
+    const int my_pos = row_pos[r], my_first = first_seen(my_pos, window);
     const float inv_cap = cap > 0.f ? 1.f / cap : 0.f;
     const float* my_bias = bias != nullptr ? bias + (size_t)(kvh * G + g0 + (r < rows ? r % gh : 0)) * L : nullptr;
     // a sink is a key of score 0 and no value that every row sees: the running maximum and sum
@@ -123,7 +123,7 @@ attn_generic_kernel(const T* q, const T* kv_pool, T* out,
             for (int c = 0; c < D; ++c) d += qr[c] * kr[c];
             d *= scale;
             const bool visible = my_pos >= 0 && j <= j_end && j <= my_pos &&
-                                 (window <= 0 || my_pos - j < window || j < keep_first);
+                                 (j >= my_first || j < keep_first);
             if (cap > 0.f) d = cap * tanhf(d * inv_cap);
             if (visible && my_bias != nullptr) d += my_bias[min(my_pos - j, L - 1)];
             s[jj] = visible ? d : -INFINITY;
@@ -183,7 +183,7 @@ static size_t attn_generic_smem(int D, int Dv) {
 TK_API int tk_attn_generic_rows() { return BM; }
 
 // q: [T, H, D]; out: [T, H, Dv]; kv_pool: [pages, 2, Hkv, P, Dp]; tiles: first token and token
-// count of each tile (tokens of one sequence, consecutive positions); window <= 0: none.
+// count of each tile (tokens of one sequence, consecutive positions); window: see first_seen.
 TK_API int tk_attn_generic(const void* q, const void* kv_pool, void* out, const int* positions,
                            const int* tok_seq, const int* block_table, int bt_stride,
                            const int* tile_tok0, const int* tile_ntok, int n_tiles,

@@ -88,14 +88,14 @@ __device__ __forceinline__ void warp_block(const uint32_t (&qf)[D / 16][4], uint
     }
     // mask: rows g (position pos_lo) and g + 8 (position pos_hi); key of element e of tile n
     if (need_mask) {
+        const int first_lo = first_seen(pos_lo, window), first_hi = first_seen(pos_hi, window);
 #pragma unroll
         for (int n = 0; n < NK / 8; ++n) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int j = j0 + n * 8 + 2 * t + (e & 1);
-                const int pos = (e < 2) ? pos_lo : pos_hi;
-                const bool visible = j <= pos && (window <= 0 || pos - j < window || j < keep_first) &&
-                                     j >= j_lo && j <= j_hi;
+                const int pos = (e < 2) ? pos_lo : pos_hi, first = (e < 2) ? first_lo : first_hi;
+                const bool visible = j <= pos && (j >= first || j < keep_first) && j >= j_lo && j <= j_hi;
                 if (!visible) s[n][e] = -INFINITY;
             }
         }
@@ -217,7 +217,7 @@ attn_prefill_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool,
     const int g = lane >> 2;
     const int pos_first = positions[tok0];
     const int pos_last = pos_first + ntok - 1;       // consecutive positions within a tile
-    const int lo = window > 0 ? max(0, pos_first - window + 1) : 0;
+    const int lo = first_seen(pos_first, window);
     const int j_begin = (lo / 64) * 64;
 
     uint32_t qf[D / 16][4];
@@ -229,6 +229,7 @@ attn_prefill_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool,
     const int w_last_row = min(rows, warp * 16 + 16) - 1;
     const int w_pos_max = w_last_row >= warp * 16 ? pos_first + w_last_row / G : -1;
     const int w_pos_min = pos_first + (warp * 16) / G;
+    const int w_first_min = first_seen(w_pos_min, window), w_first_max = first_seen(w_pos_max, window);
 
     // (a sink is a key of score 0 without a value: the running maximum and sum start from it;
     // the sum is kept in four parts, one per thread of a row)
@@ -290,9 +291,9 @@ attn_prefill_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool,
         range(it, j0, j_lo, j_hi);
         const bool kept = it < n_keep;
         const bool active = kept ? w_pos_max >= 0
-                                 : w_pos_max >= j0 && (window <= 0 || j0 + 63 > w_pos_min - window || j0 < keep_first);
+                                 : w_pos_max >= j0 && (j0 + 63 >= w_first_min || j0 < keep_first);
         if (active) {
-            const bool need_mask = kept || (j0 + 63 > w_pos_min) || (window > 0 && j0 <= w_pos_max - window) ||
+            const bool need_mask = kept || (j0 + 63 > w_pos_min) || j0 < w_first_max ||
                                    pos_lo < 0 || pos_hi < 0;
             const uint32_t base = smem + (uint32_t)(it & 1) * 2 * TILE_BYTES;
             if (keep_first > 0)
@@ -363,7 +364,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool,
     const int* bt_row = block_table + (size_t)seq * bt_stride;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, t = lane & 3;
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_seen(pos, window);
     const int j_begin = (lo / 32) * 32;
     // the key tiles: first those of the kept positions before the window, [0, keep_end), then
     // from the window's start to the token's own position
@@ -599,7 +600,7 @@ __global__ void __launch_bounds__(128) attn_decode_fused_kernel(const DecodeFuse
     const int* bt_row = a.block_table + (size_t)seq * a.bt_stride;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, t = lane & 3;
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_seen(pos, window);
     const int j_begin = (lo / 32) * 32;
     // the key tiles: first those of the kept positions before the window, [0, keep_end), then
     // from the window's start to the token's own position

@@ -145,7 +145,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int pos_first = positions[tok0];
     const int pos_last = pos_first + ntok - 1;       // consecutive positions within a tile
-    const int lo = window > 0 ? max(0, pos_first - window + 1) : 0;
+    const int lo = first_seen(pos_first, window);
     const int j_begin = (lo / AT_KEYS) * AT_KEYS;
     // Up to `max_split` CTAs (blockIdx.y) share a tile's keys, as many as leave each at least
     // AT_SPLIT_TILES key tiles: CTA `split` takes key tiles split, split + nsplit, ...; the ones
@@ -301,7 +301,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
         const int quarter = warp & 3;
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const int pos_r = r < rows ? pos_first + r / G : -1;
-        const int lo_r = window > 0 ? pos_r - window + 1 : 0;
+        const int lo_r = first_seen(pos_r, window), lo_last = first_seen(pos_last, window);
         const float scale_log2 = scale * LOG2E;
         float m_ref = -INFINITY;
         float2 l_run = make_float2(0.f, 0.f), l_alt = make_float2(0.f, 0.f);   // the row sum in four lanes
@@ -327,7 +327,7 @@ attn_prefill_tc_kernel(const __nv_bfloat16* q, const __nv_bfloat16* pool, __nv_b
             if (lane == 0) mbar_arrive(s_free(b));
             // a tile every row of the CTA sees whole needs no comparisons
             const bool kept = X && split + j * nsplit < n_keep;
-            const bool masked = j0 + AT_KEYS - 1 > pos_first || (window > 0 && j0 < pos_last - window + 1) ||
+            const bool masked = j0 + AT_KEYS - 1 > pos_first || j0 < lo_last ||
                                 rows < AT_ROWS || kept;
             // what this row sees of the tile: [see_lo, see_hi], and below keep_first whatever the window
             const int see_hi = X ? min(pos_r, tile_hi(j)) : pos_r;
@@ -567,7 +567,7 @@ TK_API int tk_attn_prefill_tc_status() {
 }
 
 // q: [T, H, 64] bfloat16; kv_pool: [pages, 2, Hkv, P, 64]; out: [T, H, 64]; tiles of at most
-// tk_attn_prefill_tc_tokens tokens of one sequence with consecutive positions; window 0 = none.
+// tk_attn_prefill_tc_tokens tokens of one sequence with consecutive positions; window: see first_seen.
 // gate: [T, >= H] bfloat16 with rows ldg apart, the per-head output gate applied to what is
 // written (null: none). nsplit > 1: up to that many CTAs share a tile's keys (alternate key tiles;
 // each tile takes as many as leave a CTA 8 key tiles), for steps with few tiles and long

@@ -175,6 +175,13 @@ __device__ __forceinline__ float2 block_sum2(float2 v, float* red) {
     return make_float2(red[64], red[65]);
 }
 
+// The first position a query at `pos` sees in a layer that does not see every earlier one: window > 0: the last `window`
+// positions; window < 0: those of its own chunk of -window positions, counted from the sequence's start; 0: all of them.
+__device__ __forceinline__ int first_seen(int pos, int window) {
+    if (window > 0) return max(0, pos - window + 1);
+    return window < 0 ? max(0, pos - pos % -window) : 0;
+}
+
 static inline int ceil_div(int a, int b) { return (a + b - 1) / b; }
 
 // ---- programmatic dependent launch -----------------------------------------------------------

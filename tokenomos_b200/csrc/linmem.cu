@@ -7,7 +7,8 @@
 //
 //   a fixed per head (a constant of the layer), a per head and token, or a per key channel and token; the last two
 //   are a = exp(-A[h] * softplus(z + bias)). beta = sigmoid(zb). With `unit`, k and q are first brought to unit
-//   length, x / sqrt(sum(x^2) + 1e-6); with `act`, q, k and v first pass silu; q is multiplied by q_scale.
+//   length, x / sqrt(sum(x^2) + 1e-6); with `act`, q, k and v first pass silu; with `freq`, the first 2 n columns of q and k
+//   are rotated by position * freq[i] (pairs (i, i + n)); q is multiplied by q_scale.
 //   Head h reads the q/k head h / (H / K).
 //
 // Eight lanes own a column of S: lane r of them has the rows 32 i + 4 r .. + 3 (i < R / 4), so that the state
@@ -48,6 +49,9 @@ struct LinMem {
     int H, K, D, V;
     float q_scale;
     int unit, act;
+    const float* freq;           // [half] or null
+    int half;
+    const int* positions;        // [T], with freq
 };
 
 __device__ __forceinline__ float lm_silu(float x) { return x / (1.0f + expf(-x)); }
@@ -151,12 +155,35 @@ __device__ __forceinline__ float lm_step(float2 (&S)[R / 2], const float* k, con
     return fmaf(kq, u, DECAY == LM_CHANNEL ? o : a * o);
 }
 
-// A warp stages one token's k and q (unit length, silu, q_scale), k . q and the decay per channel. A lane holds the
-// elements lane + 32 j.
+// A warp stages one token's k and q (silu, rotation, unit length, q_scale), k . q and the decay per channel. A lane holds
+// the elements lane + 32 j. cs: cos and sin of the token's angles (null: no rotation).
 template <typename T, int DPL>
-__device__ __forceinline__ void lm_fetch(const LinMem& m, int row, int h, int lane, float (&kv)[DPL], float (&qv)[DPL]) {
+__device__ __forceinline__ void lm_fetch(const LinMem& m, int row, int h, int lane, const float2* cs, float (&kv)[DPL],
+                                         float (&qv)[DPL]) {
     const T* src = (const T*)m.qkv + (size_t)row * m.stride;
     const int kh = h / (m.H / m.K);
+    if (cs != nullptr) {
+        // (an element's partner may be another lane's: read once more)
+        auto at = [&](int off, int d) {
+            const float x = to_f<T>(src[off + kh * m.D + d]);
+            return m.act ? lm_silu(x) : x;
+        };
+#pragma unroll
+        for (int j = 0; j < DPL; ++j) {
+            const int d = lane + 32 * j;
+            kv[j] = d < m.D ? at(m.k_off, d) : 0.f;
+            qv[j] = d < m.D ? at(m.q_off, d) : 0.f;
+            if (d < 2 * m.half) {
+                const bool low = d < m.half;
+                const int other = low ? d + m.half : d - m.half;
+                const float2 c = cs[low ? d : other];
+                const float s = low ? -c.y : c.y;
+                kv[j] = kv[j] * c.x + at(m.k_off, other) * s;
+                qv[j] = qv[j] * c.x + at(m.q_off, other) * s;
+            }
+        }
+        return;
+    }
 #pragma unroll
     for (int j = 0; j < DPL; ++j) {
         const int d = lane + 32 * j;
@@ -167,7 +194,7 @@ __device__ __forceinline__ void lm_fetch(const LinMem& m, int row, int h, int la
 template <int DPL>
 __device__ __forceinline__ void lm_shape(const LinMem& m, int lane, float (&kv)[DPL], float (&qv)[DPL], float* ks, float* qs,
                                          float* kq) {
-    if (m.act) {
+    if (m.act && m.freq == nullptr) {
 #pragma unroll
         for (int j = 0; j < DPL; ++j) {
             kv[j] = lm_silu(kv[j]);
@@ -212,14 +239,21 @@ template <typename T, int DPL, int RULE, int DECAY>
 __global__ void __launch_bounds__(256)
 linmem_prepare_kernel(const LinMem m, const LinMemPrep p) {
     constexpr int DP = 32 * DPL;
-    extern __shared__ float kq_s[];                      // [K]
+    extern __shared__ __align__(8) float prep_s[];       // cos and sin [half][2], k . q [K]
+    float2* cs = reinterpret_cast<float2*>(prep_s);
+    float* kq_s = prep_s + 2 * m.half;
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (m.freq != nullptr) {
+        const float pos = (float)m.positions[t];
+        for (int i = threadIdx.x; i < m.half; i += 256) sincosf(pos * m.freq[i], &cs[i].y, &cs[i].x);
+        __syncthreads();
+    }
     for (int kh = warp; kh < m.K; kh += 8) {
         float kv[DPL], qv[DPL];
         float* dst = p.kq + ((size_t)kh * p.rows + t) * 2 * DP;
-        lm_fetch<T, DPL>(m, t, kh * (m.H / m.K), lane, kv, qv);
+        lm_fetch<T, DPL>(m, t, kh * (m.H / m.K), lane, m.freq != nullptr ? cs : nullptr, kv, qv);
         lm_shape<DPL>(m, lane, kv, qv, dst, dst + DP, kq_s + kh);
     }
     const T* v = (const T*)m.qkv + (size_t)t * m.stride + m.v_off;
@@ -357,6 +391,7 @@ linmem_token_kernel(const LinMem m) {
     constexpr int DPL = R / 4, DP = 8 * R;
     __shared__ __align__(16) float ks[DP], qs[DP], gs[DECAY == LM_CHANNEL ? DP : 4];
     __shared__ float kq_s;
+    __shared__ float2 cs[DP / 2];
     pdl_launch_dependents();
     pdl_wait();
     const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -387,7 +422,12 @@ linmem_token_kernel(const LinMem m) {
         if (t > 0) __syncthreads();
         if (warp == 0) {
             float kv[DPL], qv[DPL];
-            lm_fetch<T, DPL>(m, row, h, lane, kv, qv);
+            if (m.freq != nullptr) {
+                const float pos = (float)m.positions[row];
+                for (int i = lane; i < m.half; i += 32) sincosf(pos * m.freq[i], &cs[i].y, &cs[i].x);
+                __syncwarp();
+            }
+            lm_fetch<T, DPL>(m, row, h, lane, m.freq != nullptr ? cs : nullptr, kv, qv);
             lm_shape<DPL>(m, lane, kv, qv, ks, qs, &kq_s);
         }
         if constexpr (DECAY == LM_CHANNEL) {
@@ -433,7 +473,8 @@ void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_c
     p.v = p.kq + (size_t)m.K * p.rows * 2 * DP;
     p.sc = reinterpret_cast<float4*>(p.v + (size_t)m.H * p.rows * p.VP);
     p.g = reinterpret_cast<float*>(p.sc + (size_t)m.H * p.rows);
-    tk_launch(linmem_prepare_kernel<T, R / 4, RULE, DECAY>, dim3(tokens), dim3(256), m.K * sizeof(float), stream, m, p);
+    tk_launch(linmem_prepare_kernel<T, R / 4, RULE, DECAY>, dim3(tokens), dim3(256),
+              (m.K + 2 * m.half) * sizeof(float), stream, m, p);
     // Two columns a thread (one where a column alone is 32 registers) in blocks of four warps; eight warps, which share
     // a stage's copies among more columns, only where even a quarter of the sequences (the least a recorded step of
     // this shape was recorded for) would fill the GPU with them
@@ -474,21 +515,25 @@ TK_API int tk_linmem_scratch(int tokens, int n_seqs, int H, int K, int D, int V,
 // qkv: [T, >= ...] rows `stride` apart holding q (K x D) at column q_off, k at k_off, v (H x V) at v_off; rule 0
 // additive, 1 delta (zb: float32 [T, >= H] rows zb_stride apart, beta's logits); decay 0 fixed (A: float32 [H], the
 // decays), 1 per head, 2 per channel (za: float32 [T, >= H] or [T, >= H D] rows za_stride apart, bias likewise one
-// row, A: float32 [H]). scratch: what tk_linmem_scratch says (16-byte aligned), null for 0. state: float32 [slots, H, V, D]; y: float32 [T, H V].
+// row, A: float32 [H]). freq (float32 [half], null: none): the rotation's frequencies, with positions [T]. scratch: what tk_linmem_scratch says (16-byte aligned), null for 0. state: float32 [slots, H, V, D]; y: float32 [T, H V].
 TK_API int tk_linmem_scan(const void* qkv, int64_t stride, int q_off, int k_off, int v_off, int rule, const float* zb,
                           int64_t zb_stride, int decay, const float* za, int64_t za_stride, const float* bias,
                           const float* A, float* state, const int* cu_seqlens, const int* seq_ctx, const int* seq_slot,
                           int n_seqs, int tokens, float* y, float* scratch, int H, int K, int D, int V, float q_scale, int unit, int act,
-                          int sm_count, int dtype, cudaStream_t stream) {
+                          const float* freq, int half, const int* positions, int sm_count, int dtype, cudaStream_t stream) {
     TK_CHECK_ARG(H > 0 && K > 0 && H % K == 0 && D > 0 && V > 0, "linear memory: %d heads over %d q/k heads", H, K);
     TK_CHECK_ARG(D <= tk_linmem_max_dim(), "linear memory: a key size of %d; up to %d are built", D, tk_linmem_max_dim());
     TK_CHECK_ARG((rule == LM_ADD && decay == LM_FIXED) || (rule == LM_DELTA && (decay == LM_HEAD || decay == LM_CHANNEL)),
                  "linear memory: rule %d with decay %d is not built", rule, decay);
     TK_CHECK_ARG(rule == LM_ADD || (zb != nullptr && za != nullptr && bias != nullptr), "linear memory: missing gates");
     TK_CHECK_ARG(n_seqs >= 0 && tokens >= 0 && A != nullptr, "linear memory: bad sizes");
+    if (freq == nullptr) half = 0;
+    TK_CHECK_ARG(half >= 0 && 2 * half <= D && (half == 0 || positions != nullptr), "linear memory: %d rotated columns of %d",
+                 2 * half, D);
+    if (half == 0) freq = nullptr;
     if (n_seqs == 0) return 0;
     const LinMem m{qkv, stride, q_off, k_off, v_off, zb, zb_stride, za, za_stride, bias, A, state, cu_seqlens, seq_ctx,
-                   seq_slot, y, H, K, D, V, q_scale, unit, act};
+                   seq_slot, y, H, K, D, V, q_scale, unit, act, freq, half, positions};
     TK_CHECK_ARG((scratch != nullptr) == (tk_linmem_scratch(tokens, n_seqs, H, K, D, V, decay) > 0),
                  "linear memory: a step of %d tokens in %d sequences without its scratch memory", tokens, n_seqs);
 #define TK_LM(TT)                                                                       \
@@ -506,7 +551,7 @@ TK_API int tk_linmem_scan(const void* qkv, int64_t stride, int q_off, int k_off,
 }
 
 // ---------------------------------------------------------------------------------------------
-// out = group_norm(y) * w * gate(z): y's row in `groups` equal parts, each divided by its own
+// out = group_norm(y) * w * gate(z) (w optional): y's row in `groups` equal parts, each divided by its own
 // sqrt(mean + eps); gate silu or sigmoid. One warp per (row, group), or, for parts longer than
 // LM_WARP_PART, one block.
 // ---------------------------------------------------------------------------------------------
@@ -553,13 +598,13 @@ norm_gate_kernel(const float* y, const T* z, int64_t z_stride, const float* __re
 #pragma unroll
     for (int k = 0; k < ITEMS; ++k) {
         const int i = lane + step * k;
-        if (i < gw) dst[i] = from_f<T>(keep[k] * rstd * w[c0 + i] * lm_gate<T>(zv[k], kind));
+        if (i < gw) dst[i] = from_f<T>(keep[k] * rstd * (w != nullptr ? w[c0 + i] : 1.0f) * lm_gate<T>(zv[k], kind));
     }
     for (int i = lane + step * ITEMS; i < gw; i += step)
-        dst[i] = from_f<T>(src[i] * rstd * w[c0 + i] * lm_gate<T>(to_f<T>(gate[i]), kind));
+        dst[i] = from_f<T>(src[i] * rstd * (w != nullptr ? w[c0 + i] : 1.0f) * lm_gate<T>(to_f<T>(gate[i]), kind));
 }
 
-// y: float32 [rows, width]; z: [rows, width] (type dtype) rows `z_stride` apart; w: float32 [width]; out: [rows, width].
+// y: float32 [rows, width]; z: [rows, width] (type dtype) rows `z_stride` apart; w: float32 [width] or null; out: [rows, width].
 TK_API int tk_norm_gate(const float* y, const void* z, int64_t z_stride, const float* w, float eps, void* out, int rows,
                         int width, int groups, int kind, int dtype, cudaStream_t stream) {
     TK_CHECK_ARG(rows >= 0 && width > 0 && groups > 0 && width % groups == 0, "norm and gate: a row of %d in %d groups",

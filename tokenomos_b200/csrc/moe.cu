@@ -1,8 +1,10 @@
 // Mixture of experts: routing, the sort of (token, expert) pairs into per-expert row blocks, a
 // grouped / batched matrix product on the CUDA cores, and the weighted combination.
 //
-//   route:   s = softmax(z[0:E]) (32-bit); the `top` largest (ties: the lowest index);
-//            w_k = s_k / (sum of the chosen s + 1e-20) * scale;  gate = sigmoid(z[E]) if the row has one
+//   route:   s = softmax(z[0:E]) (32-bit); the `top` largest choice scores (ties: the lowest index);
+//            w_k = s_k / (sum of the chosen s + 1e-20) * scale, or s_k * scale;  gate = sigmoid(z[E]) if the row has one.
+//            An expert's choice score is s, or s + correction; with groups, E / groups neighbours each, only experts of
+//            the `keep` groups with the largest choice score in them can be chosen
 //   sort:    pairs (token, k) grouped by expert, every expert's block padded to whole tiles of
 //            `tile` rows, so that a tile of the product belongs to one expert
 //   product: C[m, :] = act(A[row(m), :] . W[g]^T), g the group of m's tile (or the batch index)
@@ -19,14 +21,18 @@ constexpr int TM = 64, TN = 64, TKK = 16, GEMM_THREADS = 256;
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* logits, int64_t ld, int tokens, int E, int top, float scale, int has_gate,
-                 int* idx_out, float* w_out, float* gate_out) {
+                 const float* __restrict__ correction, int groups, int keep, int renorm, int* idx_out, float* w_out,
+                 float* gate_out) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * ROUTE_WARPS + warp;
     if (t >= tokens) return;
-    float* z = smem + (size_t)warp * E;
+    // the scores (times their sum), the choice scores (the same without a correction and groups), the groups' largest
+    const bool own = correction != nullptr || groups > 1;
+    float* z = smem + (size_t)warp * (own ? 2 * E + groups : E);
+    float* choice = own ? z + E : z;
     const float* row = logits + (size_t)t * ld;
     float mx = -INFINITY;
     for (int e = lane; e < E; e += 32) {
@@ -43,7 +49,27 @@ moe_route_kernel(const float* logits, int64_t ld, int tokens, int E, int top, fl
         sum += p;
     }
     sum = warp_sum(sum);
+    if (own)
+        for (int e = lane; e < E; e += 32) choice[e] = z[e] / sum + (correction != nullptr ? correction[e] : 0.f);
     __syncwarp();
+    if (groups > 1) {
+        float* best_of = z + 2 * E;
+        const int n = E / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float best = -INFINITY;
+            for (int e = 0; e < n; ++e) best = fmaxf(best, choice[g * n + e]);
+            best_of[g] = best;
+        }
+        __syncwarp();
+        // a group stays if fewer than `keep` groups come before it (ties: the lowest index first)
+        for (int g = lane; g < groups; g += 32) {
+            int before = 0;
+            for (int o = 0; o < groups; ++o) before += best_of[o] > best_of[g] || (best_of[o] == best_of[g] && o < g);
+            if (before >= keep)
+                for (int e = 0; e < n; ++e) choice[g * n + e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float chosen_sum = 0.f;
     float my_w = 0.f;                               // lane k keeps the k-th chosen score
     int my_e = 0;
@@ -51,7 +77,7 @@ moe_route_kernel(const float* logits, int64_t ld, int tokens, int E, int top, fl
         float best = -INFINITY;
         int at = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float v = z[e];
+            const float v = choice[e];
             if (v > best) { best = v; at = e; }     // ascending e: the lowest index of equal values stays
         }
 #pragma unroll
@@ -61,29 +87,34 @@ moe_route_kernel(const float* logits, int64_t ld, int tokens, int E, int top, fl
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
         if (at == 0x7fffffff) { at = k < E ? k : 0; best = 0.f; }    // nothing comparable: stay inside the table
-        if (lane == 0) z[at] = -INFINITY;
+        const float s = (own ? z[at] : best) / sum;
         __syncwarp();
-        const float s = best / sum;
+        if (lane == 0) choice[at] = -INFINITY;
+        __syncwarp();
         chosen_sum += s;
         if (lane == (k & 31)) { my_w = s; my_e = at; }
     }
     if (lane < top) {
         idx_out[(size_t)t * top + lane] = my_e;
-        w_out[(size_t)t * top + lane] = my_w / (chosen_sum + 1e-20f) * scale;
+        w_out[(size_t)t * top + lane] = renorm ? my_w / (chosen_sum + 1e-20f) * scale : my_w * scale;
     }
     if (has_gate && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-row[E]));
 }
 
+// correction: float32 [E] or null; groups 1: every expert can be chosen; renorm: the weights over their sum.
 TK_API int tk_moe_route(const float* logits, int64_t ld, int tokens, int E, int top, float scale, int has_gate,
-                        int* idx_out, float* w_out, float* gate_out, cudaStream_t stream) {
+                        const float* correction, int groups, int keep, int renorm, int* idx_out, float* w_out, float* gate_out, cudaStream_t stream) {
     TK_CHECK_ARG(tokens >= 0 && E > 0 && top > 0 && top <= E && top <= MAX_TOP, "moe_route: %d of %d experts (at most %d)",
                  top, E, MAX_TOP);
-    TK_CHECK_ARG((size_t)E * ROUTE_WARPS * 4 <= 48 * 1024, "moe_route: %d experts do not fit shared memory", E);
+    TK_CHECK_ARG(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top,
+                 "moe_route: %d experts out of %d of %d groups of %d", top, keep, groups, E / max(groups, 1));
+    const size_t per_warp = correction != nullptr || groups > 1 ? 2 * (size_t)E + groups : E;
+    TK_CHECK_ARG(per_warp * ROUTE_WARPS * 4 <= 48 * 1024, "moe_route: %d experts do not fit shared memory", E);
     TK_CHECK_ARG(ld >= E + (has_gate ? 1 : 0), "moe_route: rows of %lld for %d experts", (long long)ld, E);
     if (tokens == 0) return 0;
     tk_launch(moe_route_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32),
-              (size_t)E * ROUTE_WARPS * sizeof(float), stream, logits, ld, tokens, E, top, scale, has_gate, idx_out,
-              w_out, gate_out);
+              per_warp * ROUTE_WARPS * sizeof(float), stream, logits, ld, tokens, E, top, scale, has_gate, correction, groups,
+              keep, renorm, idx_out, w_out, gate_out);
     TK_CHECK_LAUNCH("moe_route");
     return 0;
 }
@@ -339,14 +370,15 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const unsigned (&a)[4], 
 // GM: rows of a tile (64: 8 warps of 32 x 32; 128: 8 warps of 64 x 32); GSTAGES: copies in flight.
 // gate (batched form only): C[g][m][:] *= sigmoid(gate[m * gate_stride + g]).
 // act 1: relu(v)^2. act 2: the weight's rows are gates and ups alternating in runs of 8; C has N / 2
-// columns, silu(gate) * up.
+// columns, silu(gate) * up. act 3: the same layout with g = min(gate, limit), u = clamp(up, -limit, limit) (limit <= 0: no
+// clamp), g * sigmoid(alpha g) * (u + shift).
 // GN: columns of a tile (128, or 64 for steps of a few rows: twice the CTAs to stream the weights).
 template <int GM, int GSTAGES, int GN>
 __global__ void __launch_bounds__(G_THREADS)
 gemm_grouped_mma_kernel(const __nv_bfloat16* A, int64_t lda, int64_t a_gs, const int* row_index,
                         const __nv_bfloat16* __restrict__ W, int64_t ldw, int64_t w_gs, const int* tile_group,
                         __nv_bfloat16* C, int64_t ldc, int64_t c_gs, int M, int N, int K, int act,
-                        const __nv_bfloat16* gate, int64_t gate_stride) {
+                        const __nv_bfloat16* gate, int64_t gate_stride, float limit, float alpha, float shift) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ __align__(16) unsigned char gsm[];
@@ -435,7 +467,7 @@ gemm_grouped_mma_kernel(const __nv_bfloat16* A, int64_t lda, int64_t a_gs, const
             const int m = m0 + wm + i * 16 + (lane >> 2) + half * 8;
             if (m >= M) continue;
             const float gv = gate != nullptr ? 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)m * gate_stride + gz]))) : 1.0f;
-            if (act == 2) {
+            if (act >= 2) {
                 // gate and up rows of the weight alternate in runs of 8: a warp's n8 blocks 2 jj and
                 // 2 jj + 1 are the gates and the ups of the same eight units, in the same lanes.
                 // Both are rounded to the storage type first, as a product that is stored would be.
@@ -446,9 +478,17 @@ gemm_grouped_mma_kernel(const __nv_bfloat16* A, int64_t lda, int64_t a_gs, const
                     float y[2];
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
-                        const float g = __bfloat162float(__float2bfloat16_rn(acc[i][2 * jj][half * 2 + e]));
-                        const float u = __bfloat162float(__float2bfloat16_rn(acc[i][2 * jj + 1][half * 2 + e]));
-                        y[e] = g / (1.f + expf(-g)) * u * gv;
+                        float g = __bfloat162float(__float2bfloat16_rn(acc[i][2 * jj][half * 2 + e]));
+                        float u = __bfloat162float(__float2bfloat16_rn(acc[i][2 * jj + 1][half * 2 + e]));
+                        if (act == 3) {
+                            if (limit > 0.f) {
+                                g = fminf(g, limit);
+                                u = fminf(fmaxf(u, -limit), limit);
+                            }
+                            y[e] = g / (1.f + expf(-alpha * g)) * (u + shift);
+                        } else {
+                            y[e] = g / (1.f + expf(-g)) * u * gv;
+                        }
                     }
                     *reinterpret_cast<__nv_bfloat162*>(C + (size_t)m * ldc + (n >> 4) * 8 + (lane & 3) * 2) =
                         __floats2bfloat162_rn(y[0], y[1]);
@@ -473,7 +513,8 @@ gemm_grouped_mma_kernel(const __nv_bfloat16* A, int64_t lda, int64_t a_gs, const
 TK_API int tk_gemm_grouped_mma(const void* A, int64_t lda, int64_t a_gs, const int* row_index, const void* W,
                                int64_t ldw, int64_t w_gs, const int* tile_group, void* C, int64_t ldc,
                                int64_t c_gs, int M, int N, int K, int groups, int act, int tile_rows,
-                               const void* gate, int64_t gate_stride, cudaStream_t stream) {
+                               const void* gate, int64_t gate_stride, float limit, float alpha, float shift,
+                               cudaStream_t stream) {
     TK_CHECK_ARG(M >= 0 && N > 0 && K > 0 && groups >= 1, "gemm_grouped_mma: bad sizes M=%d N=%d K=%d", M, N, K);
     TK_CHECK_ARG(tile_rows == 64 || tile_rows == 128, "gemm_grouped_mma: tiles of %d rows; 64 or 128", tile_rows);
     TK_CHECK_ARG(gate == nullptr || tile_group == nullptr, "gemm_grouped_mma: the row gate belongs to the batched form");
@@ -482,7 +523,7 @@ TK_API int tk_gemm_grouped_mma(const void* A, int64_t lda, int64_t a_gs, const i
                  "gemm_grouped_mma: K, N and the strides must be whole 16-byte chunks");
     TK_CHECK_ARG(((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0 && ((uintptr_t)C % 4) == 0,
                  "gemm_grouped_mma: operands must be 16-byte aligned");
-    TK_CHECK_ARG(act == 0 || act == 1 || (act == 2 && N % 16 == 0), "gemm_grouped_mma: activation %d with %d columns", act, N);
+    TK_CHECK_ARG(act == 0 || act == 1 || ((act == 2 || act == 3) && N % 16 == 0), "gemm_grouped_mma: activation %d with %d columns", act, N);
     if (M == 0) return 0;
     // few row tiles (a step of a few tokens streams the weights): columns in tiles of 64, so that
     // twice as many CTAs share the stream and an SM holds four of them
@@ -498,7 +539,8 @@ TK_API int tk_gemm_grouped_mma(const void* A, int64_t lda, int64_t a_gs, const i
                              (int)smem);                                                                            \
         tk_launch(gemm_grouped_mma_kernel<GMV, ST, GNV>, grid, dim3(G_THREADS), smem, stream,                       \
                   (const __nv_bfloat16*)A, lda, a_gs, row_index, (const __nv_bfloat16*)W, ldw, w_gs, tile_group,    \
-                  (__nv_bfloat16*)C, ldc, c_gs, M, N, K, act, (const __nv_bfloat16*)gate, gate_stride);             \
+                  (__nv_bfloat16*)C, ldc, c_gs, M, N, K, act, (const __nv_bfloat16*)gate, gate_stride, limit,       \
+                  alpha, shift);                                                                                    \
     } while (0)
     if (narrow) TK_GG(64, 6, 64);
     else if (tile_rows == 64) TK_GG(64, 5, 128);

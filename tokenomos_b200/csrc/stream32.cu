@@ -9,7 +9,7 @@
 
 // ---------------------------------------------------------------------------------------------
 // stream' = stream + x + rows + vec  (each addend optional, added in this order, 32-bit);
-// y = T(stream' * rsqrt(mean(stream'^2) + eps) * w)   (w optional: without it only the adds)
+// y = T(stream' * rsqrt(mean(stream'^2) + eps) * w)   (w optional: without it y, if there is one, is T(stream'))
 // One block per row. A thread keeps its elements of the row in registers when the row is short
 // enough (ITEMS per thread), else it reads its own writes back from stream_out.
 // ---------------------------------------------------------------------------------------------
@@ -37,6 +37,7 @@ stream32_add_norm_kernel(const float* stream_in, const T* x, int64_t x_stride, c
         for (int k = 0; k < ITEMS; ++k) {
             const int i = threadIdx.x + k * blockDim.x;
             keep[k] = i < width ? sum_at(i) : 0.f;
+            if (w == nullptr && y != nullptr && i < width) y[r * width + i] = from_f<T>(keep[k]);
             ss += keep[k] * keep[k];
         }
         if (w == nullptr) return;
@@ -53,6 +54,7 @@ stream32_add_norm_kernel(const float* stream_in, const T* x, int64_t x_stride, c
     } else {
         for (int i = threadIdx.x; i < width; i += blockDim.x) {
             const float v = sum_at(i);
+            if (w == nullptr && y != nullptr) y[r * width + i] = from_f<T>(v);
             ss += v * v;
         }
         if (w == nullptr) return;
@@ -105,6 +107,7 @@ stream32_add_norm_vec_kernel(const float* stream_in, const T* x, int64_t x_strid
                 v = make_float4(v.x + d.x, v.y + d.y, v.z + d.z, v.w + d.w);
             }
             if (stream_out != nullptr) *reinterpret_cast<float4*>(stream_out + r * width + i) = v;
+            if (w == nullptr && y != nullptr) Quad<T>::store(y + r * width + i, v);
         }
         keep[k] = v;
         ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
@@ -520,7 +523,7 @@ TK_API int tk_stream32_group_norm(const float* stream_in, const void* x, int64_t
 // ---------------------------------------------------------------------------------------------
 // The stream's add behind a norm of what is added, with the norm that reads the stream next:
 //   stream' = stream + x / sqrt(mean(x^2) + eps_x) * wx        (stream optional: zeros)
-//   y = T(stream' / sqrt(mean(stream'^2) + eps) * w)           (w optional: only the add)
+//   y = T(stream' / sqrt(mean(stream'^2) + eps) * w)           (w optional: without it y, if there is one, is T(stream'))
 // wx carries whatever multiplies the normed rows (a residual factor). One block per row; the row stays in registers
 // where it is short enough (ITEMS steps of 4 elements with VEC, of one without), else x and the stream's own writes
 // are read again.
@@ -557,6 +560,7 @@ stream32_post_norm_kernel(const float* stream_in, const T* x, int64_t x_stride, 
                 a[k] = make_float4(fmaf(b[k].x * rx, g.x, a[k].x), fmaf(b[k].y * rx, g.y, a[k].y),
                                    fmaf(b[k].z * rx, g.z, a[k].z), fmaf(b[k].w * rx, g.w, a[k].w));
                 *reinterpret_cast<float4*>(stream_out + r * width + i) = a[k];
+                if (w == nullptr && y != nullptr) Quad<T>::store(y + r * width + i, a[k]);
             }
             ss += a[k].x * a[k].x + a[k].y * a[k].y + a[k].z * a[k].z + a[k].w * a[k].w;
         }
@@ -582,6 +586,7 @@ stream32_post_norm_kernel(const float* stream_in, const T* x, int64_t x_stride, 
         for (int i = threadIdx.x; i < width; i += blockDim.x) {
             const float v = fmaf(to_f<T>(x[r * x_stride + i]) * rx, wx[i], stream_in != nullptr ? stream_in[r * width + i] : 0.f);
             stream_out[r * width + i] = v;
+            if (w == nullptr && y != nullptr) y[r * width + i] = from_f<T>(v);
             ss = fmaf(v, v, ss);
         }
         if (w == nullptr) return;
@@ -611,7 +616,7 @@ static void launch_post_norm(const float* stream_in, const void* x, int64_t x_st
 }
 
 // stream_in / stream_out: float [rows, width] (may be the same buffer; stream_in may be null); x: T rows `x_stride`
-// elements apart; wx, w: float [width] (w null: the add alone, no y).
+// elements apart; wx, w: float [width] (w null: y, if given, is the new stream's rows in T).
 TK_API int tk_stream32_post_norm(const float* stream_in, const void* x, int64_t x_stride, const float* wx, float eps_x,
                                  const float* w, float eps, float* stream_out, void* y, int rows, int width, int dtype,
                                  cudaStream_t stream) {

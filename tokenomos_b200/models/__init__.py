@@ -19,6 +19,7 @@ from tokenomos_b200.models.fakelorn import Fakelorn
 from tokenomos_b200.models.laposun import Laposun
 from tokenomos_b200.models.lfm3 import Lfm3
 from tokenomos_b200.models.lisorax import Lisorax
+from tokenomos_b200.models.namesun import Namesun
 from tokenomos_b200.models.tifisun import Tifisun
 from tokenomos_b200.parts import build_model
 from tokenomos_b200.parts.registry import Runtime, Tuning
@@ -101,3 +102,4 @@ register(Laposun())
 register(Lisorax())
 register(Fakelorn())
 register(Tifisun())
+register(Namesun())

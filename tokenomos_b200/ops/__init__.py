@@ -257,7 +257,9 @@ def attention(q: torch.Tensor, kv_pool: torch.Tensor, positions: torch.Tensor,
               scale: float, keep_first: int = 0, sink: bool = False, v_dim: int | None = None,
               round_p: bool = True, cap: float = 0.0, bias: torch.Tensor | None = None) -> torch.Tensor:
     """Causal (optionally windowed) attention of ``q`` [T, H, D] over the paged cache
-    ``kv_pool`` [pages, 2, Hkv, P, Dp], which already holds this step's keys. Tiles name runs of
+    ``kv_pool`` [pages, 2, Hkv, P, Dp], which already holds this step's keys. ``window``: here and in the other attention
+    functions the last that many positions are seen, or, negative, those of the query's own chunk of that many positions
+    counted from the sequence's start (None or 0: every earlier one). Tiles name runs of
     at most ``tokens_per_tile`` tokens of one sequence. ``keep_first``: that many first positions
     of a sequence stay visible behind the window; ``sink``: one is added to the softmax's
     denominator; ``v_dim``: the values' size (default: the keys'; the cache rows hold at least
@@ -327,13 +329,14 @@ def rotary_write(qkv: torch.Tensor, kv_pool: torch.Tensor | None, freq: torch.Te
 
 def stream32_add_norm(stream: torch.Tensor | None, x: torch.Tensor | None, weight: torch.Tensor | None,
                       eps: float, rows_add: torch.Tensor | None = None, vec_add: torch.Tensor | None = None,
-                      out_dtype: torch.dtype | None = None, in_place: bool = False, wide: bool = False):
+                      out_dtype: torch.dtype | None = None, in_place: bool = False, wide: bool = False,
+                      rows_out: bool = False):
     """A residual stream kept in 32-bit: ``stream' = stream + x + rows_add + vec_add`` (each
     optional, ``stream`` float32 [rows, width], ``x`` and ``rows_add`` in the model's storage type,
     ``vec_add`` float32 [width]) and ``y = rmsnorm(stream') * weight`` in ``out_dtype`` (default: the
     type of ``x`` / ``rows_add``), rounded once. Returns ``(y, stream')``; ``y`` is None without
     ``weight``. ``in_place``: ``stream'`` overwrites ``stream``. ``wide``: the normed rows also unrounded, in
-    float32: returns ``(y, y32, stream')``."""
+    float32: returns ``(y, y32, stream')``. ``rows_out``: without ``weight``, ``y`` is ``stream'`` itself, rounded."""
     _cuda(stream, x, weight, rows_add, vec_add)
     ref = x if x is not None else (rows_add if rows_add is not None else stream)
     if ref is None:
@@ -350,7 +353,7 @@ def stream32_add_norm(stream: torch.Tensor | None, x: torch.Tensor | None, weigh
         raise KernelError("stream32_add_norm: rows_add must be contiguous")
     w = _f32vec(weight, "norm weight", width)
     v = _f32vec(vec_add, "vec_add", width)
-    y = torch.empty(rows, width, dtype=store, device=ref.device) if w is not None else None
+    y = torch.empty(rows, width, dtype=store, device=ref.device) if w is not None or rows_out else None
     out = stream if (in_place and stream is not None) else torch.empty(rows, width, dtype=torch.float32,
                                                                     device=ref.device)
     if store not in (torch.float32, torch.bfloat16):
@@ -1053,11 +1056,15 @@ def head_gate_transpose(x: torch.Tensor, gate: torch.Tensor | None) -> torch.Ten
 
 # ---- mixture of experts --------------------------------------------------------------------------
 
-def moe_route(logits: torch.Tensor, experts: int, top: int, scale: float, has_gate: bool):
+def moe_route(logits: torch.Tensor, experts: int, top: int, scale: float, has_gate: bool,
+              correction: torch.Tensor | None = None, groups: tuple[int, int] | None = None, renorm: bool = True):
     """From float32 router rows ``[T, >= experts (+ 1)]``: the ``top`` experts of the largest
     softmax scores (int32 [T, top]), their scores over their sum times ``scale`` (float32 [T, top]),
-    and ``sigmoid`` of column ``experts`` (float32 [T]) when ``has_gate``."""
-    _cuda(logits)
+    and ``sigmoid`` of column ``experts`` (float32 [T]) when ``has_gate``. ``correction`` (float32 [experts]) joins the
+    scores for the choice only; ``groups`` (count, keep): the experts form ``count`` equal groups of neighbours and only
+    those of the ``keep`` groups with the largest choice score can be chosen; ``renorm`` False: the weights are the chosen
+    scores times ``scale``, not over their sum."""
+    _cuda(logits, correction)
     if logits.dtype != torch.float32 or logits.stride(1) != 1:
         raise KernelError("moe_route: router rows are float32 with contiguous columns")
     T = logits.shape[0]
@@ -1065,7 +1072,8 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, scale: float, has_ga
     w = torch.empty(T, top, dtype=torch.float32, device=logits.device)
     gate = torch.empty(T, dtype=torch.float32, device=logits.device) if has_gate else None
     _lib.call("tk_moe_route", _ptr(logits), logits.stride(0), T, int(experts), int(top), float(scale),
-              int(bool(has_gate)), _ptr(idx), _ptr(w), _ptr(gate), _stream())
+              int(bool(has_gate)), _ptr(_f32vec(correction, "correction", experts)), *(int(g) for g in (groups or (1, 1))),
+              int(bool(renorm)), _ptr(idx), _ptr(w), _ptr(gate), _stream())
     return idx, w, gate
 
 
@@ -1112,29 +1120,31 @@ def gemm_grouped_tiles(a_dtype: torch.dtype, n: int, k: int, rows: int) -> int:
 
 
 def gemm_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, row_index: torch.Tensor | None,
-                 rows: int, act: bool | str = False, tile: int = 64) -> torch.Tensor:
+                 rows: int, act: bool | str = False, tile: int = 64, clamp: tuple | None = None) -> torch.Tensor:
     """``out[m] = act(a[row_index[m]] @ w[g].T)`` with ``g = tile_group[m // tile]``; ``w`` [G, N, K];
     a row index of -1 reads zeros, a tile group of -1 is skipped (its rows are not written). ``act``
     True: ``relu(v)^2``; ``"swiglu8"`` (tensor-core form only, see ``gemm_grouped_fuses_swiglu``): the
     rows of ``w[g]`` are gate and up rows alternating in runs of 8 and ``out`` [rows, N / 2] is
-    ``silu(gate) * up``."""
+    ``silu(gate) * up``; ``"clamped8"``: the same with ``glu_clamped``'s activation, ``clamp`` being its (limit, alpha,
+    shift)."""
     _cuda(a, w, tile_group, row_index)
     G, N, K = w.shape
     if a.dtype != w.dtype or a.stride(1) != 1 or not w.is_contiguous() or a.shape[1] != K:
         raise KernelError(f"gemm_grouped: a {tuple(a.shape)} {a.dtype} against w {tuple(w.shape)} {w.dtype}")
-    if act == "swiglu8":
+    if act in ("swiglu8", "clamped8"):
+        limit, alpha, shift = clamp if act == "clamped8" else (None, 1.0, 0.0)
         if not gemm_grouped_fuses_swiglu(a, w):
             raise KernelError("gemm_grouped: the gated activation in the epilogue is the tensor-core form's")
         out = torch.empty(rows, N // 2, dtype=a.dtype, device=a.device)
         _lib.call("tk_gemm_grouped_mma", _ptr(a), a.stride(0), 0, _ptr(row_index), _ptr(w), K, N * K,
-                  _ptr(_i32(tile_group, "tile_group")), _ptr(out), N // 2, 0, rows, N, K, G, 2, int(tile), None, 0,
-                  _stream())
+                  _ptr(_i32(tile_group, "tile_group")), _ptr(out), N // 2, 0, rows, N, K, G, 3 if act == "clamped8" else 2, int(tile),
+                  None, 0, float(limit or 0.0), float(alpha), float(shift), _stream())
         return out
     out = torch.empty(rows, N, dtype=a.dtype, device=a.device)
     if _grouped_mma_ok(a, w, N, K):
         _lib.call("tk_gemm_grouped_mma", _ptr(a), a.stride(0), 0, _ptr(row_index), _ptr(w), K, N * K,
                   _ptr(_i32(tile_group, "tile_group")), _ptr(out), N, 0, rows, N, K, G, int(bool(act)), int(tile),
-                  None, 0, _stream())
+                  None, 0, 0.0, 1.0, 0.0, _stream())
         return out
     if tile != _lib.call("tk_gemm_grouped_tile"):
         raise KernelError(f"gemm_grouped: tiles of {tile} rows are the tensor-core form's")
@@ -1178,7 +1188,7 @@ def gemm_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = No
             raise KernelError("gemm_batched: the gate is bfloat16 [M, G] with contiguous columns")
         _lib.call("tk_gemm_grouped_mma", _ptr(a), a.stride(1), a.stride(0), None, _ptr(w), w.stride(1), w.stride(0),
                   None, _ptr(out), out.stride(1), out.stride(0), M, N, K, G, 0, 64 if M <= 64 else 128, _ptr(gate),
-                  gate.stride(0) if gate is not None else 0, _stream())
+                  gate.stride(0) if gate is not None else 0, 0.0, 1.0, 0.0, _stream())
         return out
     if gate is not None:
         raise KernelError("gemm_batched: the row gate needs the tensor-core form (bfloat16, 16-byte chunks)")
@@ -1537,10 +1547,11 @@ def stream32_group_norm(stream: torch.Tensor | None, x: torch.Tensor | None, gat
 
 
 def stream32_post_norm(stream: torch.Tensor | None, x: torch.Tensor, post_weight: torch.Tensor, post_eps: float,
-                       weight: torch.Tensor | None, eps: float, in_place: bool = False):
+                       weight: torch.Tensor | None, eps: float, in_place: bool = False, rows_out: bool = False):
     """``stream' = stream + x / sqrt(mean(x^2) + post_eps) * post_weight`` in 32-bit (``stream`` None: zeros; the weight
     carries whatever factor the normed rows get), ``y = rmsnorm(stream') * weight`` rounded once to ``x``'s type.
-    Returns ``(y, stream')``; ``y`` None without ``weight``. ``in_place``: ``stream`` is updated instead of copied."""
+    Returns ``(y, stream')``; ``y`` None without ``weight``, or, with ``rows_out``, ``stream'`` itself rounded to ``x``'s type.
+    ``in_place``: ``stream`` is updated instead of copied."""
     _cuda(stream, x, post_weight, weight)
     rows, width = x.shape
     if x.stride(1) != 1:
@@ -1548,7 +1559,7 @@ def stream32_post_norm(stream: torch.Tensor | None, x: torch.Tensor, post_weight
     if stream is not None and (stream.dtype != torch.float32 or not stream.is_contiguous() or tuple(stream.shape) != (rows, width)):
         raise KernelError("stream32_post_norm: the stream is a contiguous float32 [rows, width] tensor")
     new = stream if (in_place and stream is not None) else torch.empty(rows, width, dtype=torch.float32, device=x.device)
-    y = torch.empty(rows, width, dtype=x.dtype, device=x.device) if weight is not None else None
+    y = torch.empty(rows, width, dtype=x.dtype, device=x.device) if weight is not None or rows_out else None
     _lib.call("tk_stream32_post_norm", _ptr(stream), _ptr(x), x.stride(0), _ptr(_f32vec(post_weight, "post-norm weight", width)),
               float(post_eps), _ptr(_f32vec(weight, "norm weight", width)), float(eps), _ptr(new), _ptr(y), rows, width,
               _dtype_code(x), _stream())
@@ -1567,20 +1578,22 @@ def linmem_scan(qkv: torch.Tensor, offsets: tuple, rule: str, decay: str, A: tor
                 cu_seqlens: torch.Tensor, seq_ctx: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, heads: int, kv_heads: int,
                 dim: int, v_dim: int, q_scale: float = 1.0, unit: bool = False, act: bool = False,
                 beta: torch.Tensor | None = None, gates: torch.Tensor | None = None, bias: torch.Tensor | None = None,
-                sm_count: int = 148) -> torch.Tensor:
+                sm_count: int = 148, freq: torch.Tensor | None = None, positions: torch.Tensor | None = None) -> torch.Tensor:
     """A matrix memory per head over a step's tokens: ``S <- a S``, then ``S <- S + k v^T`` (``rule`` "add") or ``u =
     sigmoid(beta) (v - S^T k), S <- S + k u^T`` ("delta"), ``y = S^T q``. ``qkv`` [T, *]: q (``kv_heads`` x dim) at column
     ``offsets[0]``, k at ``offsets[1]``, v (``heads`` x v_dim) at ``offsets[2]``; head h reads q/k head ``h / (heads /
     kv_heads)``. ``decay``: "fixed" (``A`` float32 [heads] holds a), "head" or "channel" (``a = exp(-A[h] softplus(gates
     + bias))`` with ``gates`` float32 [T, >= heads] or [T, >= heads dim]). ``act``: q, k
-    and v pass silu first; ``unit``: q and k are brought to unit length; q is multiplied by ``q_scale``. ``state`` float32
+    and v pass silu first; ``freq`` (float32): the first ``2 len(freq)`` columns of q and k are rotated by ``positions *
+    freq`` (pairs (i, i + len(freq))); ``unit``: q and k are brought to unit length; q is multiplied by ``q_scale``. ``state`` float32
     [slots, heads, v_dim, dim]. Returns ``y`` float32 [T, heads v_dim]."""
-    _cuda(qkv, A, state, beta, gates, bias)
+    _cuda(qkv, A, state, beta, gates, bias, freq, positions)
     T = qkv.shape[0]
     if qkv.stride(1) != 1:
         raise KernelError("linmem_scan: rows of q, k and v with contiguous columns")
     if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, v_dim, dim) or not state.is_contiguous():
         raise KernelError(f"linmem_scan: the state is float32 [slots, {heads}, {v_dim}, {dim}]")
+    half = freq.numel() if freq is not None else 0
     cols = {"fixed": 0, "head": heads, "channel": heads * dim}[decay]
     for name, t, need in (("beta", beta, heads if rule == "delta" else 0), ("gates", gates, cols)):
         if need and (t is None or t.dtype != torch.float32 or t.stride(1) != 1 or t.shape[0] != T or t.shape[1] < need):
@@ -1594,13 +1607,14 @@ def linmem_scan(qkv: torch.Tensor, offsets: tuple, rule: str, decay: str, A: tor
               gates.stride(0) if gates is not None else 0, _ptr(_f32vec(bias, "decay bias", cols)) if cols else None,
               _ptr(_f32vec(A, "A", heads)), _ptr(state), _ptr(_i32(cu_seqlens, "cu_seqlens")), _ptr(_i32(seq_ctx, "seq_ctx")),
               _ptr(_i32(seq_slot, "seq_slot")), int(n_seqs), T, _ptr(y), _ptr(scratch), heads, kv_heads, dim, v_dim,
-              float(q_scale), int(bool(unit)), int(bool(act)), int(sm_count), _dtype_code(qkv), _stream())
+              float(q_scale), int(bool(unit)), int(bool(act)), _ptr(_f32vec(freq, "freq", half)) if half else None, half,
+              _ptr(_i32(positions, "positions")) if half else None, int(sm_count), _dtype_code(qkv), _stream())
     return y
 
 
-def norm_gate(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, gate: str) -> torch.Tensor:
+def norm_gate(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor | None, eps: float, groups: int, gate: str) -> torch.Tensor:
     """Each of the row's ``groups`` equal parts of ``y`` (float32 [T, C]) divided by its own ``sqrt(mean + eps)``, times
-    ``weight`` [C], times ``gate(z)`` ("silu" or "sigmoid"; ``z`` [T, C] in the storage type, rows may be strided)."""
+    ``weight`` [C] (None: ones), times ``gate(z)`` ("silu" or "sigmoid"; ``z`` [T, C] in the storage type, rows may be strided)."""
     _cuda(y, z, weight)
     T, C = y.shape
     if y.dtype != torch.float32 or not y.is_contiguous() or z.stride(1) != 1 or tuple(z.shape) != (T, C):
@@ -1651,6 +1665,36 @@ def qkv_row_norm_write(qkv: torch.Tensor, wq: torch.Tensor, wk: torch.Tensor | N
     return q
 
 
+def qkv_head_norm_write(qkv: torch.Tensor, wq: torch.Tensor | None, wk: torch.Tensor | None, eps: float,
+                        positions: torch.Tensor, tok_seq: torch.Tensor, block_table: torch.Tensor | None,
+                        pool: torch.Tensor | None, heads: int, kv_heads: int, dim: int, v_dim: int,
+                        other: torch.Tensor | None = None, lam: float = 0.0) -> torch.Tensor:
+    """From rows ``[q | k | v]`` the queries [T, heads, dim] and, in ``pool`` [pages, 2, kv_heads, P, row] at each token's
+    position, the keys and values; every q head and every k head is RMS-normed (times ``wq`` / ``wk`` [dim] if given).
+    ``other`` [T, kv_heads v_dim] (rows may be strided): the values are ``(1 - lam) v + lam other``. ``pool`` None: queries
+    only."""
+    _cuda(qkv, wq, wk, positions, tok_seq, block_table, pool, other)
+    T = qkv.shape[0]
+    need = heads * dim + (kv_heads * (dim + v_dim) if pool is not None else 0)
+    if qkv.stride(1) != 1 or qkv.shape[1] < need:
+        raise KernelError(f"qkv_head_norm_write: rows of at least {need} contiguous columns")
+    if other is not None and (other.dtype != qkv.dtype or other.stride(1) != 1 or tuple(other.shape) != (T, kv_heads * v_dim)):
+        raise KernelError(f"qkv_head_norm_write: the other values are {qkv.dtype} [{T}, {kv_heads * v_dim}] with contiguous columns")
+    q = torch.empty(T, heads, dim, dtype=qkv.dtype, device=qkv.device)
+    P = dp = bt = 0
+    if pool is not None:
+        if (pool.dtype != qkv.dtype or not pool.is_contiguous() or pool.dim() != 5 or pool.shape[1] != 2
+                or pool.shape[2] != kv_heads):
+            raise KernelError(f"qkv_head_norm_write: the pool is {qkv.dtype} [pages, 2, {kv_heads}, P, row]")
+        P, dp, bt = pool.shape[3], pool.shape[4], _i32(block_table, "block_table").stride(0)
+    _lib.call("tk_qkv_head_norm_write", _ptr(qkv), qkv.stride(0), _ptr(_f32vec(wq, "q norm weight", dim)),
+              _ptr(_f32vec(wk, "k norm weight", dim)), float(eps), _ptr(other), other.stride(0) if other is not None else 0,
+              1.0 - float(lam), float(lam), _ptr(_i32(positions, "positions")), _ptr(_i32(tok_seq, "tok_seq")),
+              _ptr(block_table), bt, _ptr(q), _ptr(pool), T, heads, max(kv_heads, 1), dim, v_dim, P, dp, _dtype_code(qkv),
+              _stream())
+    return q
+
+
 def attention_biased_mma_supported(heads: int, kv_heads: int, head_dim: int, v_dim: int, row: int,
                                    dtype: torch.dtype) -> bool:
     """Whether ``attention_biased_mma`` takes the shape (bfloat16, sizes in multiples of 8 up to 128, at most 16 query
@@ -1667,13 +1711,14 @@ def attention_biased_mma(q: torch.Tensor, kv_pool: torch.Tensor, out: torch.Tens
                          tok_seq: torch.Tensor, block_table: torch.Tensor, tile_tok0: torch.Tensor | None,
                          tile_ntok: torch.Tensor | None, singles: torch.Tensor | None, n_single: int, nsplit: int,
                          window: int | None, scale: float, cap: float = 0.0, bias_log2: torch.Tensor | None = None,
-                         bounded: bool = False) -> None:
+                         bounded: bool = False, sink: bool = False) -> None:
     """Softmax attention with scores ``cap tanh(q.k scale / cap) + bias[h, min(i - j, L - 1)]`` on the tensor cores
     (``bias_log2`` is ``bias`` over ``ln 2``): the
     tiles of prompt portions (``attention_biased_mma_tokens`` tokens each) and ``n_single`` single tokens (their rows
     in ``singles``; None: rows 0 .. n_single - 1), each shared ``nsplit`` ways over its keys. ``q`` [T, H, D], ``out``
-    [T, H, Dv], ``kv_pool`` [pages, 2, Hkv, P, row]. ``bounded``: cap and bias keep every score, in base-2 logarithms,
-    well inside a float's exponents, so the softmax needs no running maximum."""
+    [T, H, Dv], ``kv_pool`` [pages, 2, Hkv, P, row]. ``bounded``: every score, in base-2 logarithms, is known to lie
+    well inside a float's exponents, so the softmax needs no running maximum; ``sink``: one is added to the softmax's
+    denominator."""
     _cuda(q, kv_pool, out, positions, tok_seq, block_table, tile_tok0, tile_ntok, singles, bias_log2)
     T, H, D = q.shape
     _, two, Hkv, P, Dp = kv_pool.shape
@@ -1691,4 +1736,4 @@ def attention_biased_mma(q: torch.Tensor, kv_pool: torch.Tensor, out: torch.Tens
               _ptr(_i32(tile_tok0, "tile_tok0")) if n_tiles else None, _ptr(_i32(tile_ntok, "tile_ntok")) if n_tiles else None,
               n_tiles, _ptr(_i32(singles, "singles")) if singles is not None else None, int(n_single), int(nsplit), _ptr(part_o),
               _ptr(part_ml), H, Hkv, D, Dv, Dp, P, int(window or 0), float(scale), float(cap or 0.0), *_bias_table(bias_log2, H),
-              int(bool(bounded)), _stream())
+              int(bool(bounded)), int(bool(sink)), _stream())

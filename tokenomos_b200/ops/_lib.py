@@ -81,12 +81,12 @@ _SIGNATURES = {
     "tk_attn_latent_mma": [P, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, I, F, I, P, P, I, P],
     "tk_attn_latent_merge": [P, P, P, I, I, I, P],
     "tk_head_gate_transpose": [P, P, L, P, I, I, I, I, P],
-    "tk_moe_route": [P, L, I, I, I, F, I, P, P, P, P],
+    "tk_moe_route": [P, L, I, I, I, F, I, P, I, I, I, P, P, P, P],
     "tk_moe_sort": [P, I, I, I, I, I, P, P, P, P, P],
     "tk_gather_rows_or_zero": [P, P, P, I, I, I, P],
     "tk_gemm_grouped_tile": [],
     "tk_gemm_grouped_simt": [P, L, L, P, P, L, L, P, P, L, L, I, I, I, I, I, I, P],
-    "tk_gemm_grouped_mma": [P, L, L, P, P, L, L, P, P, L, L, I, I, I, I, I, I, P, L, P],
+    "tk_gemm_grouped_mma": [P, L, L, P, P, L, L, P, P, L, L, I, I, I, I, I, I, P, L, F, F, F, P],
     "tk_moe_combine": [P, P, P, P, P, P, I, I, I, I, P],
     "tk_relu2": [P, L, I, P],
     "tk_scale_rows_f32": [P, L, P, F, I, I, I, P],
@@ -111,12 +111,13 @@ _SIGNATURES = {
     "tk_gemm_skinny_gelu": [P, L, P, L, P, P, L, I, I, I, I, P],
     "tk_linmem_max_dim": [],
     "tk_linmem_scratch": [I, I, I, I, I, I, I],
-    "tk_linmem_scan": [P, L, I, I, I, I, P, L, I, P, L, P, P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, I, I, I, P],
+    "tk_linmem_scan": [P, L, I, I, I, I, P, L, I, P, L, P, P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, I, P, I, P, I, I, P],
     "tk_norm_gate": [P, P, L, P, F, P, I, I, I, I, I, P],
     "tk_pair_norm_mean": [P, L, P, L, P, P, F, F, P, I, I, I, P],
     "tk_attn_biased_mma_supported": [I, I, I, I, I],
     "tk_attn_biased_mma_tokens": [I, I],
-    "tk_attn_biased_mma": [P, P, P, P, P, P, I, P, P, I, P, I, I, P, P, I, I, I, I, I, I, I, F, F, P, I, I, P],
+    "tk_attn_biased_mma": [P, P, P, P, P, P, I, P, P, I, P, I, I, P, P, I, I, I, I, I, I, I, F, F, P, I, I, I, P],
+    "tk_qkv_head_norm_write": [P, L, P, P, F, P, L, F, F, P, P, P, I, P, P, I, I, I, I, I, I, I, I, P],
     "tk_qkv_row_norm_write": [P, L, P, P, F, P, P, P, I, P, P, I, I, I, I, I, I, I, I, P],
 }
 

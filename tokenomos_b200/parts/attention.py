@@ -19,7 +19,9 @@ a bias by distance ``- r1[h] ln(1 + r2[h] (i - j))`` and a query temperature ``1
 / every) + 1)``; ``PointwiseWeights``); ``diff`` (differential attention, ``DiffMaps``: every head has two
 softmax maps over the same values, each with its own half of the query and of the key, joined as
 ``a_1 - lambda a_2`` and brought to unit root mean square per head); ``shape`` (``ScoreShape``: the scores' soft cap ``c tanh(s / c)`` and,
-after it, a learned bias by distance). A position part may keep state per request (a short
+after it, a learned bias by distance); ``chunk`` (in place of a window: a query sees the keys of its own chunk of that many
+positions, counted from the sequence's start, up to its own); ``value_mix`` (``ValueMix``: the cached values are mixed
+with an earlier layer's values of the same token). A position part may keep state per request (a short
 convolution on q, k and v): it then has ``state_specs()`` and is called with the layer's ``call``.
 """
 
@@ -32,7 +34,7 @@ from dataclasses import dataclass
 import torch
 
 from tokenomos_b200 import ops
-from tokenomos_b200.parts.contract import HeadLayout, PagedKV, SharedState, StepContext, WindowKV
+from tokenomos_b200.parts.contract import ChunkKV, HeadLayout, PagedKV, SharedState, StepContext, ValueRows, WindowKV
 from tokenomos_b200.parts.linear import Linear
 from tokenomos_b200.parts.registry import DEFAULT_TUNING, Runtime, Tuning, builder_of, register
 
@@ -85,6 +87,15 @@ class ScoreShape:
         return (2.0 * self.cap + 2.0 * reach) / math.log(2.0) <= 100.0
 
 
+@dataclass(frozen=True)
+class ValueMix:
+    """``v <- (1 - lam) v + lam v_first``, with ``v_first`` what entry ``source`` of the layer list projected as its values of the
+    same token (before any mix); ``source`` None: this layer is where they come from, and keeps its own."""
+
+    source: int | None
+    lam: float = 0.0
+
+
 def distance_bucket(n: int, rows: int, far: float) -> int:
     """The row of a ``rows``-row table of biases for distance ``n``: the first half one by one, the second half in equal
     steps of the logarithm up to ``far``."""
@@ -102,7 +113,8 @@ class Attention:
                  gate_fused: bool = False, tuning: Tuning = DEFAULT_TUNING, sink: bool = False,
                  keep_first: int = 0, v_dim: int | None = None, v_is_k: bool = False,
                  gate_kind: str = "head", exact: bool = False, pointwise: PointwiseWeights | None = None,
-                 diff: DiffMaps | None = None, shape: ScoreShape | None = None):
+                 diff: DiffMaps | None = None, shape: ScoreShape | None = None, chunk: int | None = None,
+                 value_mix: ValueMix | None = None):
         """``gate``: the per-head gate's projection as a part of its own; ``gate_fused``: its rows
         are the last of ``qkv``'s instead (after q, k, v, then zero rows up to a multiple of 8), so
         that one product yields both. With ``diff``, ``heads`` counts the maps (twice the output heads)
@@ -133,6 +145,16 @@ class Attention:
             self.shape_bounded = shape.bounded          # (asked once: it reads the bias from the device)
             # the tensor-core kernels carry scores in base-2 logarithms
             self.bias_log2 = (shape.bias.double() / math.log(2.0)).float() if shape.bias is not None else None
+        self.chunk, self.value_mix = chunk, value_mix
+        if chunk is not None and (chunk < 1 or window is not None or pointwise is not None or diff is not None or keep_first
+                                  or (shape is not None and shape.bias is not None)):
+            raise ValueError("attention: chunks stand in place of a window, under a plain softmax without a bias by distance")
+        if value_mix is not None and (kv_source is not None or v_is_k or not getattr(rope, "takes_value_mix", False)):
+            raise ValueError("attention: mixed values need a projection and a cache of their own and a position part that "
+                             "writes them")
+        # how far back a query sees, as the kernels take it (``ops.attention``), and how many keys that is at most
+        self.reach = -chunk if chunk is not None else window
+        self.span = chunk if chunk is not None else window
         if pointwise is not None and (sink or keep_first):
             raise ValueError("attention: a sink and kept first positions belong to the softmax")
         # what the one-kernel decode form and the norms folded into the projections do not take
@@ -140,7 +162,10 @@ class Attention:
         # kernel takes everything)
         self.extended = bool(self.sink or self.keep_first or self.v_is_k or v_dim != head_dim
                              or gate_kind != "head" or self.exact or pointwise is not None or diff is not None
-                             or shape is not None)
+                             or shape is not None or chunk is not None or value_mix is not None)
+        # queries and keys brought to unit root mean square per head bound every score by head_dim * scale
+        self.scores_bounded = (getattr(rope, "head_norm", False) and q_norm is None and k_norm is None and self.shape is None
+                               and 2.0 * head_dim * abs(scale if scale is not None else head_dim ** -0.5) / math.log(2.0) <= 100.0)
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads over {kv_heads} KV heads")
         if head_dim > ops.ATTENTION_MAX_HEAD_DIM:
@@ -182,6 +207,8 @@ class Attention:
         if self.kv_source is not None:
             return {"kv": SharedState(self.kv_source, "kv"), **more}
         row = max(self.head_dim, self.v_dim)         # a cache row holds a key or a value
+        if self.chunk is not None:
+            return {"kv": ChunkKV(self.kv_heads, row, self.chunk), **more}
         if self.window is None:
             return {"kv": PagedKV(self.kv_heads, row), **more}
         return {"kv": WindowKV(self.kv_heads, row, self.window, self.keep_first), **more}
@@ -297,8 +324,9 @@ class Attention:
             q = self.rope.encode_qk(qkv, ctx, self.head_layout, pool if own_kv else None,
                                     table if own_kv else None, call=call)
         else:
+            more = {"mix": self._value_rows(qkv, ctx, call)} if self.value_mix is not None else {}
             q = self.rope.encode_qk(qkv, ctx, self.head_layout, pool if own_kv else None,
-                                    table if own_kv else None)
+                                    table if own_kv else None, **more)
         if self.pointwise is not None:
             out = self._attend_pointwise(q, pool, table, ctx)
             if gate is not None and self.gate_kind == "head":
@@ -313,22 +341,38 @@ class Attention:
             elif gate is not None:
                 ops.sigmoid_gate(out, gate)
             return out
-        # the tensor-core kernels take everything but value heads of another size than the keys
+        # the tensor-core kernels take everything but value heads of another size than the keys, which another one
+        # takes where no first positions are kept
         if self.v_dim == self.head_dim and ops.attention_mma_supported(self.heads, self.kv_heads, self.head_dim,
                                                                        q.dtype):
             return self._attend_mma(q, pool, table, ctx, gate)
+        if not self.keep_first and self._biased_supported(pool, q):
+            out = self._attend_biased(q, pool, table, ctx, 0.0, None, self.scores_bounded)
+            if gate is not None and self.gate_kind == "head":
+                ops.head_gate(out, gate, self.heads, self.v_dim)
+            elif gate is not None:
+                ops.sigmoid_gate(out, gate)
+            return out
         rows = ops.attention_rows()
         group = self.heads // self.kv_heads
         per_tile = max(1, rows // group)
         _, tok0, _, ntok = ctx.tiles(per_tile)
         out = ops.attention(q, pool, ctx.positions, ctx.tok_seq, table, tok0, ntok, per_tile,
-                            self.window, self.scale, self.keep_first, self.sink, self.v_dim,
+                            self.reach, self.scale, self.keep_first, self.sink, self.v_dim,
                             round_p=not self.exact)
         if gate is not None and self.gate_kind == "head":
             ops.head_gate(out, gate, self.heads, self.v_dim)
         elif gate is not None:
             ops.sigmoid_gate(out, gate)
         return out
+
+    def _value_rows(self, qkv: torch.Tensor, ctx: StepContext, call: int) -> ValueRows | None:
+        """What this step's values are mixed with; the layer they come from leaves its rows for the step's later layers."""
+        if self.value_mix.source is not None:
+            return ValueRows(ctx.scratch[("values", self.value_mix.source)], self.value_mix.lam)
+        first = (self.heads + self.kv_heads) * self.head_dim
+        ctx.scratch[("values", call)] = qkv[:, first:first + self.kv_heads * self.v_dim]
+        return None
 
     # whether pointwise weights may take the tensor-core kernels (TOKENOMOS_B200_ATTN_POINT_MMA=0: never)
     pointwise_mma = os.environ.get("TOKENOMOS_B200_ATTN_POINT_MMA", "1") != "0"
@@ -377,28 +421,33 @@ class Attention:
         sizes (bfloat16), prompt portions in tiles of 64 rows and single tokens shared out over their keys; else the
         general kernel."""
         sh = self.shape
-        T = q.shape[0]
-        if self.biased_mma and ops.attention_biased_mma_supported(self.heads, self.kv_heads, self.head_dim, self.v_dim,
-                                                                  pool.shape[-1], q.dtype):
-            out = torch.empty(T, self.heads, self.v_dim, dtype=q.dtype, device=q.device)
-            tok0 = ntok = singles = None
-            n_single, nsplit = ctx.n_tokens, 1
-            if not ctx.host.decode_only:
-                _, tok0, _, ntok = ctx.tiles(ops.attention_biased_mma_tokens(self.heads, self.kv_heads), "multi")
-                singles = ctx.singles()
-                n_single = singles.numel()
-            if n_single:
-                longest = ctx.host.longest
-                if self.window is not None:
-                    longest = min(longest, self.window)
-                nsplit = self.decode_splits(n_single, self.kv_heads, longest, self.tuning)
-            ops.attention_biased_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, singles, n_single, nsplit,
-                                     self.window, self.scale, sh.cap, self.bias_log2, self.shape_bounded)
-            return out
+        if self._biased_supported(pool, q):
+            return self._attend_biased(q, pool, table, ctx, sh.cap, self.bias_log2, self.shape_bounded)
         per_tile = max(1, ops.attention_rows() // (self.heads // self.kv_heads))
         _, tok0, _, ntok = ctx.tiles(per_tile)
-        return ops.attention(q, pool, ctx.positions, ctx.tok_seq, table, tok0, ntok, per_tile, self.window, self.scale,
+        return ops.attention(q, pool, ctx.positions, ctx.tok_seq, table, tok0, ntok, per_tile, self.reach, self.scale,
                              v_dim=self.v_dim, round_p=not self.exact, cap=sh.cap, bias=sh.bias)
+
+    def _biased_supported(self, pool, q) -> bool:
+        return self.biased_mma and ops.attention_biased_mma_supported(self.heads, self.kv_heads, self.head_dim, self.v_dim,
+                                                                      pool.shape[-1], q.dtype)
+
+    def _attend_biased(self, q, pool, table, ctx: StepContext, cap: float, bias_log2, bounded: bool) -> torch.Tensor:
+        out = torch.empty(q.shape[0], self.heads, self.v_dim, dtype=q.dtype, device=q.device)
+        tok0 = ntok = singles = None
+        n_single, nsplit = ctx.n_tokens, 1
+        if not ctx.host.decode_only:
+            _, tok0, _, ntok = ctx.tiles(ops.attention_biased_mma_tokens(self.heads, self.kv_heads), "multi")
+            singles = ctx.singles()
+            n_single = singles.numel()
+        if n_single:
+            longest = ctx.host.longest
+            if self.span is not None:
+                longest = min(longest, self.span)
+            nsplit = self.decode_splits(n_single, self.kv_heads, longest, self.tuning)
+        ops.attention_biased_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, singles, n_single, nsplit,
+                                 self.reach, self.scale, cap, bias_log2, bounded, self.sink)
+        return out
 
     # whether prompt portions may take the tcgen05 kernel (TOKENOMOS_B200_ATTN_TC=0: never)
     prefill_tc = os.environ.get("TOKENOMOS_B200_ATTN_TC", "1") != "0"
@@ -459,22 +508,22 @@ class Attention:
         _, tok0, _, ntok = ctx.tiles(per_tile, "multi")
         if tok0.numel() and tc:
             nsplit = self.prefill_splits(ctx.n_tokens, tok0.numel(), per_tile, self.kv_heads, self.tuning)
-            ops.attention_prefill_tc(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, self.window,
+            ops.attention_prefill_tc(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, self.reach,
                                      self.scale, gate, nsplit, self.keep_first, self.sink, by_element)
         elif tok0.numel():
-            ops.attention_prefill_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, self.window,
+            ops.attention_prefill_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, tok0, ntok, self.reach,
                                       self.scale, gate, self.keep_first, self.sink, by_element)
         # every sequence brings one token: row i is sequence i's, no list of rows needed
         decode_only = ctx.host.decode_only
         singles = None if decode_only else ctx.singles()
         if decode_only or singles.numel():
             longest = ctx.host.longest
-            if self.window is not None:
-                longest = min(longest, self.window)
+            if self.span is not None:
+                longest = min(longest, self.span)
             rows = ctx.n_tokens if decode_only else singles.numel()
             nsplit = self.decode_splits(rows, self.kv_heads, longest, self.tuning)
             ops.attention_decode_mma(q, pool, out, ctx.positions, ctx.tok_seq, table, singles,
-                                     self.window, self.scale, nsplit, gate, self.keep_first, self.sink, by_element)
+                                     self.reach, self.scale, nsplit, gate, self.keep_first, self.sink, by_element)
         return out
 
 
@@ -525,6 +574,15 @@ def _shape(params: dict | None, tensors: dict, heads: int, window: int | None) -
     return ScoreShape(float(params.get("cap") or 0.0), bias)
 
 
+def _value_mix(params: dict | None, tensors: dict) -> ValueMix | None:
+    """``params``: ``source`` (an earlier entry of the layer list, or None: this layer's values are the ones others mix in);
+    tensor ``v_mix``: lambda, one number (not read where the values come from)."""
+    if params is None:
+        return None
+    source = params.get("source")
+    return ValueMix(source, 0.0 if source is None else float(tensors["v_mix"].double()))
+
+
 @register("mixer", "attention")
 def build_attention(params: dict, tensors: dict, rt: Runtime) -> Attention:
     rope_spec = params["position"]
@@ -559,4 +617,5 @@ def build_attention(params: dict, tensors: dict, rt: Runtime) -> Attention:
         keep_first=params.get("keep_first", 0), v_dim=params.get("v_dim"), v_is_k=v_is_k,
         gate_kind=params.get("gate_kind", "head"), exact=params.get("exact", False),
         pointwise=_pointwise(params.get("pointwise"), tensors), diff=_diff(params.get("diff"), tensors),
-        shape=_shape(params.get("shape"), tensors, params["heads"], params.get("window")))
+        shape=_shape(params.get("shape"), tensors, params["heads"], params.get("window")), chunk=params.get("chunk"),
+        value_mix=_value_mix(params.get("value_mix"), tensors))

@@ -11,7 +11,8 @@ State memory comes in two shapes:
 - paged, growing with the sequence: ``PagedKV`` (every position kept) and ``WindowKV`` (only the
   last ``window`` positions are ever read, and with ``keep_first`` the first positions of the
   sequence as well; pages behind the window, but for those that hold kept positions, are given
-  back). Specs with equal ``group`` share one pool's page numbering and one block table per
+  back) and ``ChunkKV`` (a query reads its own chunk of ``chunk`` positions; a chunk's pages are
+  given back when the sequence leaves it). Specs with equal ``group`` share one pool's page numbering and one block table per
   request;
 - fixed size per request: ``SlotState``, a row ``[*shape]`` of a ``[slots, *shape]`` tensor,
   row 0 being the null row that padded sequences point at. A request that starts at position
@@ -24,7 +25,8 @@ A spec says what the cache manager has to do for it through three attributes, so
 bring a spec class of its own: ``storage`` (``"paged"``, ``"slot"`` or ``"shared"``); for paged
 storage ``group`` (specs with equal groups share page numbers and block tables), ``window``
 (None: every position is kept), optionally ``keep_first`` (positions at the start of a sequence
-that a window never passes) and ``page_shape(page_size)`` (the shape of one page); for slot
+that a window never passes), ``chunk`` (positions are read chunk by chunk; ``window`` is then a
+chunk's size) and ``page_shape(page_size)`` (the shape of one page); for slot
 storage ``shape`` and ``dtype``; for shared storage ``source`` and ``name``.
 
 Captured steps. With ``graphs=True`` the engine records a step's kernels once per shape and
@@ -83,6 +85,28 @@ class WindowKV:
 
 
 @dataclass(frozen=True)
+class ChunkKV:
+    """Keys and values that are read chunk by chunk: a query at position i reads the positions of its
+    own chunk, ``floor(j / chunk) == floor(i / chunk)``, counted from the sequence's start."""
+
+    kv_heads: int
+    head_dim: int
+    chunk: int
+    storage = "paged"
+
+    @property
+    def window(self) -> int:
+        return self.chunk
+
+    @property
+    def group(self) -> tuple:
+        return ("chunk", self.chunk)
+
+    def page_shape(self, page_size: int) -> tuple[int, ...]:
+        return (2, self.kv_heads, page_size, self.head_dim)
+
+
+@dataclass(frozen=True)
 class LatentKV:
     """One row ``[row]`` per position instead of keys and values per head: ``[pages, page, row]``
     (a compressed key/value latent and whatever rides with it). ``window`` None: every position
@@ -119,7 +143,7 @@ class SharedState:
 
 
 # the specs the framework's own parts use; any object with the attributes above is one too
-StateSpec = PagedKV | WindowKV | LatentKV | SlotState | SharedState
+StateSpec = PagedKV | WindowKV | ChunkKV | LatentKV | SlotState | SharedState
 # the "call" under which the state of a model's embedding part is keyed (it is no entry of the
 # layer list)
 EMBED_CALL = -1
@@ -254,6 +278,15 @@ class HeadLayout:
     v_is_k: bool = False
 
 
+@dataclass(frozen=True)
+class ValueRows:
+    """Another layer's values of the step's tokens ([T, kv_heads v_dim], before any mix) and the weight they get:
+    the values that are cached are ``(1 - lam) v + lam rows``."""
+
+    rows: torch.Tensor
+    lam: float
+
+
 @runtime_checkable
 class PositionEncoding(Protocol):
     """Owns everything between the fused q/k/v projection and attention over the cache: how
@@ -278,3 +311,6 @@ class PositionEncoding(Protocol):
     # (attention does, in steps where every sequence brings one token) instead of calling
     # ``encode_qk``; both ways give the same bits. Encodings without the method are always
     # called through ``encode_qk``.
+    #
+    # Optional. An encoding that writes values mixed with another layer's (``encode_qk(..., mix=ValueRows)``)
+    # says so with ``takes_value_mix = True``.

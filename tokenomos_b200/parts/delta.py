@@ -1,4 +1,4 @@
-"""Linear memories with a fixed-size state per request: the gated delta rule and lightning attention.
+"""Linear memories with a fixed-size state per request: the gated delta rule, lightning attention and retention.
 
 ``GatedDelta`` (kind ``delta_rule``): per head a matrix S [dim, v_dim] from zero,
 
@@ -11,7 +11,9 @@
     out = W_o (headnorm(o) * w * gate),   gate = silu(W_g h), or sigmoid(W_g2 (W_g1 h))      (w shared by the heads)
 
 ``LightningMemory`` (kind ``lightning``): ``q, k, v = silu(W h)``, ``S <- decay[head] S + k v^T``, ``o = S^T q``, the
-concatenated heads RMS-normed together, times ``w * sigmoid(W_g h)``, through ``W_o``.
+concatenated heads RMS-normed together, times ``w * sigmoid(W_g h)``, through ``W_o``. Kind ``retention``: the same
+recurrence without the silu on q, k and v, with a rotation of q and k by position, ``k`` times ``dim^(-1/2)``, every head's
+``o`` RMS-normed on its own (no weight) and the gate ``silu(W_g h)``.
 
 The states, everything that enters a recurrence after the projections and convolutions (beta and the decays from
 products with a 32-bit result, unit lengths), and the norms are 32-bit whatever the storage type. Both parts read the
@@ -26,6 +28,7 @@ from tokenomos_b200 import ops
 from tokenomos_b200.parts.contract import SlotState, StepContext
 from tokenomos_b200.parts.linear import Linear
 from tokenomos_b200.parts.registry import Runtime, register
+from tokenomos_b200.parts.rope import Rotary
 
 
 def padded_rows(w: torch.Tensor, to: int = 8) -> torch.Tensor:
@@ -130,9 +133,13 @@ def build_gated_delta(params: dict, tensors: dict, rt: Runtime) -> GatedDelta:
 class LightningMemory:
     capture_safe = True
 
-    def __init__(self, in_proj: Linear, out_proj: Linear, decay: list[float], norm: torch.Tensor, heads: int, dim: int,
-                 v_dim: int, eps: float):
-        """``in_proj``: the rows of q, k (heads x dim each), v and the output gate (heads x v_dim each)."""
+    def __init__(self, in_proj: Linear, out_proj: Linear, decay: list[float], norm: torch.Tensor | None, heads: int, dim: int,
+                 v_dim: int, eps: float, act: bool = True, q_scale: float = 1.0, freq: torch.Tensor | None = None,
+                 norm_groups: int = 1, gate: str = "sigmoid"):
+        """``in_proj``: the rows of q, k (heads x dim each), v and the output gate (heads x v_dim each). ``act``: q, k and v pass
+        silu; ``q_scale``: a factor on q (one on k is the same number in every output); ``freq``: the frequencies of a
+        rotate-half rotation of q's and k's first columns; ``norm_groups``: equal parts of the output row that are normed on
+        their own; ``norm`` None: no weight; ``gate``: silu or sigmoid."""
         self.in_proj, self.out_proj = in_proj, out_proj
         self.heads, self.dim, self.v_dim, self.eps = int(heads), int(dim), int(v_dim), float(eps)
         if self.dim > ops.LINMEM_MAX_DIM:
@@ -143,8 +150,13 @@ class LightningMemory:
         if (in_proj.out_features != 2 * self.heads * (self.dim + self.v_dim)
                 or out_proj.in_features != self.heads * self.v_dim):
             raise ValueError("lightning attention: the projections do not match the head sizes")
-        self.norm = norm.float().reshape(-1).contiguous()
-        self.decay = torch.tensor([float(d) for d in decay], dtype=torch.float32, device=self.norm.device)
+        if gate not in ops.GATE_KINDS or (freq is not None and 2 * freq.numel() > self.dim):
+            raise ValueError(f"linear memory: gate {gate!r}, rotation of {2 * freq.numel() if freq is not None else 0} of {self.dim} "
+                             "columns")
+        self.norm = norm.float().reshape(-1).contiguous() if norm is not None else None
+        self.act, self.q_scale, self.freq = bool(act), float(q_scale), freq
+        self.norm_groups, self.gate = int(norm_groups), gate
+        self.decay = torch.tensor([float(d) for d in decay], dtype=torch.float32, device=in_proj.weight.device)
         self.sm_count = in_proj.tuning.sm_count
 
     def state_specs(self) -> dict:
@@ -159,9 +171,10 @@ class LightningMemory:
     def forward_projected(self, proj: torch.Tensor, ctx: StepContext, call: int) -> torch.Tensor:
         H, D, V = self.heads, self.dim, self.v_dim
         y = ops.linmem_scan(proj, (0, H * D, 2 * H * D), "add", "fixed", self.decay, ctx.states[(call, "S")], ctx.cu_seqlens,
-                            ctx.seq_ctx, ctx.seq_slot, ctx.n_seqs, H, H, D, V, act=True, sm_count=self.sm_count)
+                            ctx.seq_ctx, ctx.seq_slot, ctx.n_seqs, H, H, D, V, q_scale=self.q_scale, act=self.act,
+                            sm_count=self.sm_count, freq=self.freq, positions=ctx.positions)
         gate = proj[:, 2 * H * D + H * V:2 * H * (D + V)]
-        return self.out_proj(ops.norm_gate(y, gate, self.norm, self.eps, 1, "sigmoid"))
+        return self.out_proj(ops.norm_gate(y, gate, self.norm, self.eps, self.norm_groups, self.gate))
 
 
 @register("mixer", "lightning")
@@ -169,3 +182,17 @@ def build_lightning_memory(params: dict, tensors: dict, rt: Runtime) -> Lightnin
     mats = [tensors[n] for n in ("q", "k", "v", "gate")]
     return LightningMemory(Linear.fused(mats, tuning=rt.tuning), Linear(tensors["o"], tuning=rt.tuning), params["decay"],
                            tensors["norm"], params["heads"], params["dim"], params["v_dim"], params["eps"])
+
+
+@register("mixer", "retention")
+def build_retention(params: dict, tensors: dict, rt: Runtime) -> LightningMemory:
+    """Tensors ``q``, ``k``, ``v``, ``gate``, ``o``; params ``heads``, ``dim``, ``v_dim``, ``decay`` (one per head), ``eps`` and ``rot``
+    (``dims``, ``base``; None: no rotation)."""
+    mats = [tensors[n] for n in ("q", "k", "v", "gate")]
+    rot, freq = params.get("rot"), None
+    if rot is not None and rot["dims"]:
+        freqs, _ = Rotary.table(rot["dims"], float(rot["base"]), None)
+        freq = torch.tensor(freqs, dtype=torch.float64).to(torch.float32).to(rt.device).contiguous()
+    return LightningMemory(Linear.fused(mats, tuning=rt.tuning), Linear(tensors["o"], tuning=rt.tuning), params["decay"], None,
+                           params["heads"], params["dim"], params["v_dim"], params["eps"], act=False,
+                           q_scale=params["dim"] ** -0.5, freq=freq, norm_groups=params["heads"], gate="silu")

@@ -1,9 +1,12 @@
 """Mixture of experts feed-forward.
 
     z = W_router h (32-bit);  s = softmax(z);  the ``top`` experts of the largest s
-    w_k = s_k / (sum of the chosen s + 1e-20) * scale
+    w_k = s_k / (sum of the chosen s + 1e-20) * scale, or s_k * scale (``RouteRule.renorm`` False)
     out = sum_k w_k * expert_k(h)  [+ sigmoid(W_sg h) * shared(h)]
-    expert(h) = W_down act(W_up h),  act(v) = relu(v)^2     (no biases)
+    expert(h) = W_down act(W_up h),  act(v) = relu(v)^2, or a gated form     (no biases)
+
+``RouteRule``: a correction per expert that joins the scores for the choice only, and groups of neighbouring experts of
+which only the best few (by their largest choice score) can be chosen from.
 
 The router (and the shared expert's gate row, appended to it) is a 32-bit matrix in any model.
 The (token, expert) pairs of a step are sorted by expert on the device into blocks of whole
@@ -15,6 +18,7 @@ launches are the same whatever the routing, so a step can be recorded.
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 
 import torch
 
@@ -23,27 +27,39 @@ from tokenomos_b200.parts.linear import Linear
 from tokenomos_b200.parts.registry import Runtime, register
 
 
+@dataclass(frozen=True)
+class RouteRule:
+    """How experts are chosen and weighed beyond the softmax: ``correction`` float32 [experts] or None; ``groups`` (count,
+    keep) or None; ``renorm``: the weights over the chosen scores' sum."""
+
+    correction: torch.Tensor | None = None
+    groups: tuple[int, int] | None = None
+    renorm: bool = True
+
+
 class RoutedExperts:
     capture_safe = True
 
     def __init__(self, router: Linear, up: torch.Tensor, down: torch.Tensor, top: int, scale: float,
                  shared_up: Linear | None = None, shared_down: Linear | None = None, shared_gate: bool = False,
-                 library_rows: int = 1024, activation: str = "relu2", shared: object | None = None):
+                 library_rows: int = 1024, activation: str = "relu2", shared: object | None = None,
+                 rule: RouteRule = RouteRule(), clamp: tuple[float | None, float, float] = (None, 1.0, 0.0)):
         """``up`` [E, ff, width], ``down`` [E, width, ff]; ``router`` [E (+ 1 if ``shared_gate``) (+ zero
         rows), width] (it may carry a bias). ``activation`` "relu2": ``act(v) = relu(v)^2``; "swiglu": an
         expert is ``W_down (silu(W_gate h) * (W_up h))`` and ``up`` holds each expert's gate rows, then its
         up rows ([E, 2 ff, width]; kept with gate and up alternating in runs of 8 where the kernels
-        take that). ``shared``: a whole feed-forward part that every token runs and whose output is added (in
+        take that); "clamped": the same layout with ``ClampedGLU``'s activation, ``clamp`` being its (limit, alpha, shift).
+        ``shared``: a whole feed-forward part that every token runs and whose output is added (in
         place of ``shared_up`` / ``shared_down``, which are the ``relu2`` form)."""
         self.shared = shared
         if shared is not None and (shared_up is not None or shared_gate):
             raise ValueError("mixture of experts: one shared expert")
-        if activation not in ("relu2", "swiglu"):
-            raise ValueError(f"mixture of experts: activation {activation!r}: 'relu2' or 'swiglu'")
-        self.activation = activation
+        if activation not in ("relu2", "swiglu", "clamped"):
+            raise ValueError(f"mixture of experts: activation {activation!r}: 'relu2', 'swiglu' or 'clamped'")
+        self.activation, self.gated, self.rule, self.clamp = activation, activation != "relu2", rule, clamp
         self.experts, self.ff, self.width = up.shape
         self.gate_run = 0
-        if activation == "swiglu":
+        if self.gated:
             self.ff //= 2
             if up.dtype == torch.bfloat16 and self.ff % 8 == 0:
                 # gate and up rows alternating in runs of 8: the tensor-core product then has a unit's
@@ -54,6 +70,10 @@ class RoutedExperts:
         self.top, self.scale = int(top), float(scale)
         if not 1 <= self.top <= self.experts:
             raise ValueError(f"mixture of experts: {self.top} of {self.experts} experts per token")
+        if rule.groups is not None:
+            count, keep = rule.groups
+            if count < 1 or self.experts % count or not 1 <= keep <= count or keep * (self.experts // count) < self.top:
+                raise ValueError(f"mixture of experts: {self.top} experts out of {keep} of {count} groups of {self.experts}")
         if tuple(down.shape) != (self.experts, self.width, self.ff):
             raise ValueError("mixture of experts: down projections do not match the up projections")
         if (shared_up is None) != (shared_down is None) or (shared_gate and shared_up is None):
@@ -71,7 +91,8 @@ class RoutedExperts:
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         z = self.router(x, out_dtype=torch.float32)
-        idx, w, gate = ops.moe_route(z, self.experts, self.top, self.scale, self.shared_gate)
+        idx, w, gate = ops.moe_route(z, self.experts, self.top, self.scale, self.shared_gate, self.rule.correction,
+                                     self.rule.groups, self.rule.renorm)
         if self.library and x.shape[0] * self.top >= self.library_rows:
             y, pair_row = self._experts_library(x, idx)
             return ops.moe_combine(y, pair_row, w, self._shared(x), gate)
@@ -80,14 +101,20 @@ class RoutedExperts:
                                       x.shape[0] * self.top)
         row_token, pair_row, tile_expert = ops.moe_sort(idx, self.experts, tile)
         rows = row_token.numel()
-        if self.activation == "swiglu" and self.gate_run and ops.gemm_grouped_fuses_swiglu(x, self.up):
-            act = ops.gemm_grouped(x, self.up, tile_expert, row_token, rows, act="swiglu8", tile=tile)
-        elif self.activation == "swiglu":
-            act = ops.swiglu(ops.gemm_grouped(x, self.up, tile_expert, row_token, rows, tile=tile), self.gate_run)
+        if self.gated and self.gate_run and ops.gemm_grouped_fuses_swiglu(x, self.up):
+            act = ops.gemm_grouped(x, self.up, tile_expert, row_token, rows, tile=tile, clamp=self.clamp,
+                                   act="swiglu8" if self.activation == "swiglu" else "clamped8")
+        elif self.gated:
+            act = self._activate(ops.gemm_grouped(x, self.up, tile_expert, row_token, rows, tile=tile))
         else:
             act = ops.gemm_grouped(x, self.up, tile_expert, row_token, rows, act=True, tile=tile)
         y = ops.gemm_grouped(act, self.down, tile_expert, None, rows, tile=tile)
         return ops.moe_combine(y, pair_row, w, self._shared(x), gate)
+
+    def _activate(self, rows: torch.Tensor) -> torch.Tensor:
+        if self.activation == "swiglu":
+            return ops.swiglu(rows, self.gate_run)
+        return ops.glu_clamped(rows, *self.clamp, self.gate_run) if self.activation == "clamped" else ops.relu2(rows)
 
     def _shared(self, x: torch.Tensor) -> torch.Tensor | None:
         if self.shared is not None:
@@ -102,8 +129,7 @@ class RoutedExperts:
         row_token, pair_row, _, ends = ops.moe_sort(idx, self.experts, 8, ends=True)
         rows = ops.gather_rows_or_zero(x, row_token)
         act = torch._grouped_mm(rows, self.up.transpose(1, 2), offs=ends)
-        act = ops.swiglu(act, self.gate_run) if self.activation == "swiglu" else ops.relu2(act)
-        return torch._grouped_mm(act, self.down.transpose(1, 2), offs=ends), pair_row
+        return torch._grouped_mm(self._activate(act), self.down.transpose(1, 2), offs=ends), pair_row
 
 
 @register("feed_forward", "relu2_moe")
@@ -150,3 +176,32 @@ def build_gated_experts(params: dict, tensors: dict, rt: Runtime) -> RoutedExper
             bias = torch.cat((bias.float(), torch.zeros(pad, dtype=torch.float32, device=bias.device)))
     return RoutedExperts(Linear(w, bias, tuning=rt.tuning), up, down, params["top"], params.get("scale", 1.0),
                          library_rows=rt.tuning.grouped_library_rows, activation="swiglu", shared=shared)
+
+
+@register("feed_forward", "clamped_moe")
+def build_clamped_experts(params: dict, tensors: dict, rt: Runtime) -> RoutedExperts:
+    """Experts with ``ClampedGLU``'s form (``limit``, ``alpha``, ``shift`` for all of them), chosen by softmax scores plus
+    ``correction`` (a tensor, optional) among the best of ``groups`` = (count, keep) (optional), weighed by the scores
+    (``renorm``: over their sum). Tensors ``shared.gate|up|down``: a shared expert of the same form with a limit of its own
+    (``shared_limit``) that every token runs, added unweighted."""
+    from tokenomos_b200.parts.ffn import build_clamped_glu
+
+    n = params["experts"]
+    form = {k: params[k] for k in ("alpha", "shift") if k in params}
+    shared = None
+    if "shared.gate" in tensors:
+        shared = build_clamped_glu({"limit": params.get("shared_limit"), **form},
+                                   {k: tensors["shared." + k] for k in ("gate", "up", "down")}, rt)
+    up = torch.stack([torch.cat((tensors[f"e{i}.gate"], tensors[f"e{i}.up"])) for i in range(n)])
+    down = torch.stack([tensors[f"e{i}.down"] for i in range(n)])
+    w = tensors["router"].to(rt.dtype)
+    pad = -n % 8
+    if pad:
+        w = torch.cat((w, w.new_zeros(pad, w.shape[1])))
+    correction = tensors.get("correction")
+    groups = params.get("groups")
+    rule = RouteRule(correction.float().reshape(-1).contiguous() if correction is not None else None,
+                     tuple(groups) if groups is not None else None, bool(params.get("renorm", True)))
+    return RoutedExperts(Linear(w, tuning=rt.tuning), up, down, params["top"], params.get("scale", 1.0),
+                         library_rows=rt.tuning.grouped_library_rows, activation="clamped", shared=shared, rule=rule,
+                         clamp=(params.get("limit"), form.get("alpha", 1.0), form.get("shift", 0.0)))

@@ -81,20 +81,27 @@ class StreamNorm32:
     own root mean square (the weight still covers the whole row). A ``GatedRows`` handed in as ``pre``
     gates what is added: ``stream' = stream + x * sigmoid(gate)``. Another ``StreamNorm32`` handed in as ``pre``
     norms what is added (a norm behind the sublayer): ``stream' = stream + mult * norm(x)`` with that norm's weight,
-    eps and ``mult``, the add and both norms in one kernel; ``mult`` belongs to a norm in that place only."""
+    eps and ``mult``, the add and both norms in one kernel; ``mult``, and a ``layer_scale`` (one more factor per column of the
+    normed rows), belong to a norm in that place only."""
 
     capture_safe = True
     stream_dtype = torch.float32
 
     def __init__(self, weight: torch.Tensor, eps: float, offset: float = 0.0,
-                 store: torch.dtype = torch.float32, groups: int = 1, mult: float = 1.0):
+                 store: torch.dtype = torch.float32, groups: int = 1, mult: float = 1.0,
+                 layer_scale: torch.Tensor | None = None):
         self.weight = (weight.float() + float(offset)).contiguous()
         self.eps = float(eps)
         self.width = weight.numel()
         self.store = store
         self.groups = int(groups)
         self.mult = float(mult)
-        self.scaled = self.weight if self.mult == 1.0 else (self.weight * self.mult).contiguous()
+        # what a norm behind a sublayer multiplies the normed rows by, as one vector
+        self.scaled = self.weight if self.mult == 1.0 else self.weight * self.mult
+        self.behind_only = self.mult != 1.0 or layer_scale is not None
+        if layer_scale is not None:
+            self.scaled = self.scaled * layer_scale.float().reshape(-1)
+        self.scaled = self.scaled.contiguous()
         if self.groups < 1 or self.width % self.groups:
             raise ValueError(f"rmsnorm32: a row of {self.width} in {groups} groups")
 
@@ -103,8 +110,8 @@ class StreamNorm32:
         be the stream itself (float32 in a 16-bit model) or the rows that start one. ``pre``: a
         ``PendingAdd``, a ``GatedRows``, the sublayer's own post-norm or None. ``wide``: the normed rows
         also unrounded: returns ``(norm(stream), the same in float32, stream)``."""
-        if self.mult != 1.0:
-            raise ValueError("rmsnorm32: a factor on the normed rows belongs to a norm behind a sublayer")
+        if self.behind_only:
+            raise ValueError("rmsnorm32: a factor or scale on the normed rows belongs to a norm behind a sublayer")
         if isinstance(pre, StreamNorm32):
             if wide or self.groups > 1 or pre.groups > 1:
                 raise ValueError("rmsnorm32: behind a sublayer's norm neither norms in groups nor unrounded rows are built")
@@ -136,9 +143,40 @@ class StreamNorm32:
 @register("norm", "rmsnorm32")
 def build_stream_norm32(params: dict, tensors: dict, rt: Runtime) -> StreamNorm32:
     norm = StreamNorm32(tensors["weight"], params["eps"], params.get("offset", 0.0), rt.dtype,
-                        params.get("groups", 1), params.get("mult", 1.0))
+                        params.get("groups", 1), params.get("mult", 1.0), tensors.get("layer_scale"))
     # taps of a convolution on what a sublayer behind this norm reads (``parts.parallel``): the
     # arrangement that has one finds them here
     norm.input_taps = tensors.get("taps")
     norm.conv_tile = rt.tuning.conv_tile
     return norm
+
+
+class StreamRows32:
+    """In the place of a norm before a sublayer where there is none: the sublayer reads the 32-bit residual stream itself,
+    rounded to the storage type. ``add_norm`` only does the add: a norm behind the sublayer before (``StreamNorm32``) and
+    the write of the new stream and of its rounded rows are one kernel."""
+
+    capture_safe = True
+    stream_dtype = torch.float32
+
+    def __init__(self, store: torch.dtype):
+        self.store = store
+
+    def add_norm(self, x: torch.Tensor, residual: torch.Tensor | None, pre=None):
+        rows_out = self.store != torch.float32           # a 32-bit model's sublayers read the stream as it is
+        if isinstance(pre, StreamNorm32):
+            y, stream = ops.stream32_post_norm(residual, x, pre.scaled, pre.eps, None, 0.0, rows_out=rows_out)
+        elif pre is not None:
+            raise ValueError("rows of a 32-bit stream: only a rmsnorm32 can be behind the sublayer before")
+        elif residual is None and x.dtype == torch.float32:          # the stream itself
+            if not rows_out:
+                return x, x
+            y, stream = ops.stream32_add_norm(x, None, None, 0.0, out_dtype=self.store, in_place=True, rows_out=True)
+        else:
+            y, stream = ops.stream32_add_norm(residual, x, None, 0.0, out_dtype=self.store, rows_out=rows_out)
+        return (y if rows_out else stream), stream
+
+
+@register("norm", "stream32")
+def build_stream_rows32(params: dict, tensors: dict, rt: Runtime) -> StreamRows32:
+    return StreamRows32(rt.dtype)

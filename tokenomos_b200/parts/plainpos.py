@@ -8,6 +8,9 @@ reads part m of both. The part hands each map to the kernels as a head of its ow
 width with zeros outside its part, so that the kernels' ``q . k`` is the map's score against keys that are
 stored once (``[T, heads, maps, dim] -> [T, heads * maps, maps * dim]``).
 
+``head_norm``: an RMS norm over every q head and every k head (with the head layout's weights, or none), in the same
+kernel as the write, which can also mix the values with another layer's (``encode_qk(..., mix=...)``).
+
 ``q_norm`` / ``k_norm``: an RMS norm over a token's whole query row and whole key row (all heads at once, before they
 are split) with weights of those sizes, in the same kernel as the write.
 """
@@ -17,7 +20,7 @@ from __future__ import annotations
 import torch
 
 from tokenomos_b200 import ops
-from tokenomos_b200.parts.contract import HeadLayout, StepContext
+from tokenomos_b200.parts.contract import HeadLayout, StepContext, ValueRows
 from tokenomos_b200.parts.registry import Runtime, register
 
 
@@ -25,17 +28,27 @@ class PlainQKV:
     capture_safe = True
 
     def __init__(self, maps: int = 1, q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None,
-                 eps: float = 0.0):
+                 eps: float = 0.0, head_norm: bool = False):
         self.maps = int(maps)
+        self.head_norm = self.takes_value_mix = bool(head_norm)
         if self.maps < 1:
             raise ValueError(f"plain q/k/v: {maps} maps")
-        if self.maps > 1 and q_norm is not None:
-            raise ValueError("plain q/k/v: norms over the whole rows go with one map a head")
+        if self.maps > 1 and (q_norm is not None or head_norm):
+            raise ValueError("plain q/k/v: norms over whole rows or heads go with one map a head")
+        if head_norm and q_norm is not None:
+            raise ValueError("plain q/k/v: norms over the whole rows or over the heads")
         self.q_norm = q_norm.float().reshape(-1).contiguous() if q_norm is not None else None
         self.k_norm = k_norm.float().reshape(-1).contiguous() if k_norm is not None else None
         self.eps = float(eps)
 
-    def encode_qk(self, qkv, ctx: StepContext, heads: HeadLayout, pool, table):
+    def encode_qk(self, qkv, ctx: StepContext, heads: HeadLayout, pool, table, mix: ValueRows | None = None):
+        if self.head_norm:
+            if heads.v_is_k:
+                raise ValueError("plain q/k/v: values that are the keys are not built here")
+            return ops.qkv_head_norm_write(
+                qkv, heads.q_norm, heads.k_norm, self.eps, ctx.positions, ctx.tok_seq, table, pool, heads.heads, heads.kv_heads,
+                heads.head_dim, heads.v_dim or heads.head_dim, mix.rows if mix is not None else None,
+                mix.lam if mix is not None else 0.0)
         if heads.q_norm is not None or heads.k_norm is not None or heads.v_is_k:
             raise ValueError("plain q/k/v: per-head norms and values that are the keys are not built here")
         if heads.heads % self.maps or heads.head_dim % self.maps:
@@ -49,4 +62,5 @@ class PlainQKV:
 
 @register("position", "plain")
 def build_plain_qkv(params: dict, tensors: dict, rt: Runtime) -> PlainQKV:
-    return PlainQKV(params.get("maps", 1), tensors.get("q_norm"), tensors.get("k_norm"), params.get("eps", 0.0))
+    return PlainQKV(params.get("maps", 1), tensors.get("q_norm"), tensors.get("k_norm"), params.get("eps", 0.0),
+                    params.get("head_norm", False))
