@@ -58,11 +58,13 @@ def attention(x: torch.Tensor, W: dict, p: str, m: dict, eps: float, first: torc
     return torch.cat(heads, -1) @ W[p + "o"].T
 
 
-def rotate(x: torch.Tensor, rot: dict) -> torch.Tensor:
+def rotate(x: torch.Tensor, rot: dict | None) -> torch.Tensor:
     """``x`` [T, heads, dim], row t at position t."""
+    if rot is None or not rot["dims"]:
+        return x
     half = rot["dims"] // 2
     i = torch.arange(half, dtype=F64)
-    a = torch.arange(x.shape[0], dtype=F64)[:, None] * float(rot["base"]) ** (-2.0 * i / max(rot["dims"], 1))
+    a = torch.arange(x.shape[0], dtype=F64)[:, None] * float(rot["base"]) ** (-2.0 * i / rot["dims"])
     c, s = torch.cos(a)[:, None], torch.sin(a)[:, None]
     u, w = x[..., :half], x[..., half:2 * half]
     return torch.cat((u * c - w * s, w * c + u * s, x[..., 2 * half:]), -1)
@@ -83,8 +85,8 @@ def retention_scan(q, k, v, decay):
 def retention(x: torch.Tensor, W: dict, p: str, m: dict, eps: float) -> torch.Tensor:
     T = x.shape[0]
     H, D, V = m["heads"], m["dim"], m["vdim"]
-    q = rotate((x @ W[p + "q"].T).reshape(T, H, D), m["rot"])
-    k = rotate((x @ W[p + "k"].T).reshape(T, H, D), m["rot"]) * D ** -0.5
+    q = rotate((x @ W[p + "q"].T).reshape(T, H, D), m.get("rot"))
+    k = rotate((x @ W[p + "k"].T).reshape(T, H, D), m.get("rot")) * D ** -0.5
     o = retention_scan(q, k, (x @ W[p + "v"].T).reshape(T, H, V), m["decay"])
     return (rms(o, eps).reshape(T, H * V) * silu(x @ W[p + "g"].T)) @ W[p + "o"].T
 

@@ -9,7 +9,7 @@ import pytest
 import torch
 
 from tokenomos_b200.cache.manager import CacheError, CacheManager, OutOfPages
-from tokenomos_b200.parts.contract import PagedKV, SharedState, SlotState, WindowKV
+from tokenomos_b200.parts.contract import ChunkKV, PagedKV, SharedState, SlotState, WindowKV
 
 SPECS = {
     (0, "conv"): SlotState((2, 8)),
@@ -53,6 +53,30 @@ def test_pages_follow_the_tokens_and_return():
     c.admit("c")
     c.extend("c", 5)
     assert c.block_table("c", ("full",)) == [1, 2] and c.slot("c") == 1   # lowest free first
+
+
+@pytest.mark.parametrize("chunk, page", [(6, 4), (8, 4), (1, 4), (3, 1), (50, 4), (5, 8)])
+def test_chunk_group_gives_a_chunk_back_when_the_sequence_leaves_it(chunk, page):
+    c = CacheManager({(0, "kv"): ChunkKV(2, 8, chunk)}, page, 60, 2, torch.float32, "meta", 200)
+    group = ("chunk", chunk)
+    assert set(c.groups) == {group} and tuple(c.states[(0, "kv")].shape) == (60, 2, 2, page, 8)
+    c.admit("a")
+    done = 0
+    for n in [1, 1, 4, 1, 7, 1, 1, 2, 9, 1, 1, 1, 13, 1, 1, 1, 1]:
+        c.extend("a", n)
+        table = c.block_table("a", group)
+        # every position a query of this step reads is held: from the first one's chunk to the last one
+        held = [b for b in range(len(table)) if table[b]]
+        assert set(range(done - done % chunk, done + n)) <= {p for b in held for p in range(b * page, (b + 1) * page)}
+        c.commit("a", n)
+        done += n
+        c.check()
+        # and nothing of a page that lies wholly before the next query's chunk
+        first = (done - done % chunk) // page
+        assert all(page_no == 0 for page_no in c.block_table("a", group)[:first])
+        assert len(c.groups[group].pages.held) == max(0, -(-done // page) - first)
+    c.release("a")
+    c.check()
 
 
 def test_window_group_gives_back_what_it_has_passed():

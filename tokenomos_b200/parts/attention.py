@@ -152,9 +152,6 @@ class Attention:
         if value_mix is not None and (kv_source is not None or v_is_k or not getattr(rope, "takes_value_mix", False)):
             raise ValueError("attention: mixed values need a projection and a cache of their own and a position part that "
                              "writes them")
-        # how far back a query sees, as the kernels take it (``ops.attention``), and how many keys that is at most
-        self.reach = -chunk if chunk is not None else window
-        self.span = chunk if chunk is not None else window
         if pointwise is not None and (sink or keep_first):
             raise ValueError("attention: a sink and kept first positions belong to the softmax")
         # what the one-kernel decode form and the norms folded into the projections do not take
@@ -200,6 +197,16 @@ class Attention:
         self.head_layout = HeadLayout(heads, own_kv, head_dim, self.q_norm,
                                       self.k_norm if own_kv else None, self.eps,
                                       v_dim=v_dim, v_is_k=self.v_is_k)
+
+    @property
+    def reach(self) -> int | None:
+        """How far back a query sees, as the kernels take it (``ops.attention``)."""
+        return -self.chunk if self.chunk is not None else self.window
+
+    @property
+    def span(self) -> int | None:
+        """The most keys a query sees (None: all before it)."""
+        return self.chunk if self.chunk is not None else self.window
 
     def state_specs(self) -> dict:
         # a position part with state of its own per request lists it (under names of its own)
@@ -341,12 +348,12 @@ class Attention:
             elif gate is not None:
                 ops.sigmoid_gate(out, gate)
             return out
-        # the tensor-core kernels take everything but value heads of another size than the keys, which another one
-        # takes where no first positions are kept
+        # the tensor-core kernels take heads of 64 and 128 with values of the keys' size; another one takes other sizes
+        # where no first positions are kept and nothing asks for the softmax's weights rounded before they are summed up
         if self.v_dim == self.head_dim and ops.attention_mma_supported(self.heads, self.kv_heads, self.head_dim,
                                                                        q.dtype):
             return self._attend_mma(q, pool, table, ctx, gate)
-        if not self.keep_first and self._biased_supported(pool, q):
+        if self.exact and not self.keep_first and self._biased_supported(pool, q):
             out = self._attend_biased(q, pool, table, ctx, 0.0, None, self.scores_bounded)
             if gate is not None and self.gate_kind == "head":
                 ops.head_gate(out, gate, self.heads, self.v_dim)
