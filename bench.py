@@ -2049,6 +2049,226 @@ def tifisun_kernels(z: dict, pk: dict) -> list[dict]:
     return rows
 
 
+# ---------------------------------------------------------------------------------------------
+# --design namesun: the Namesun decoder beside Fakelorn (the other design with a recurrent state per head, attention that
+# looks back a fixed distance, experts with a shared one and a 32-bit stream) at equal sizes
+# ---------------------------------------------------------------------------------------------
+
+_NS2048 = dict(width=2048, layers=8, heads=16, kv_heads=4, dim=128, att_heads=16, att_kv=4, att_dim=128, att_vdim=128, chunk=1024, window=1024, ret_heads=16, ret_dim=128,
+               ret_vdim=128, ff=6144, experts=32, top=4, groups=8, keep=4, expert_ff=1024, shared_ff=2048, vocab=65536)
+NAMESUN_SIZES = {
+    "width2048": _NS2048,
+    "width2048_v64": dict(_NS2048, att_vdim=64),
+    "width1024": dict(_NS2048, width=1024, dim=64, att_dim=64, att_vdim=64, ret_dim=64, ret_vdim=64, ff=4096, experts=16, groups=4, keep=3,
+                      top=4, expert_ff=512, shared_ff=1024),
+}
+
+
+def namesun_config(z: dict) -> dict:
+    """Groups of four layers: attention with a dense feed-forward, two of retention and one of attention with experts."""
+    att = {"type": "attention", "mixer": {"heads": z["att_heads"], "kv_heads": z["att_kv"], "dim": z["att_dim"],
+                                          "vdim": z["att_vdim"], "scale": z["att_dim"] ** -0.5, "mask": {"size": z["chunk"]},
+                                          "v_mix": True}}
+    ret = {"type": "retention", "mixer": {"heads": z["ret_heads"], "dim": z["ret_dim"], "vdim": z["ret_vdim"],
+                                          "decay": [1.0 - 2.0 ** (-5.0 - 0.5 * h) for h in range(z["ret_heads"])],
+                                          "rot": {"base": 10000.0, "dims": z["ret_dim"]}}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": z["groups"], "keep": z["keep"]}},
+           "shared": {"ff": z["shared_ff"], "limit": 7.0}}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    layers = [dict(att if i % 4 in (0, 3) else ret, mlp=dense if i % 4 == 0 else moe) for i in range(z["layers"])]
+    return {"architecture": "Namesun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "layers": layers}
+
+
+def namesun_like_config(z: dict) -> dict:
+    """Fakelorn at the same sizes: state-space layers of the same state where Namesun has retention, differential attention
+    of the same heads and cache over a window of a chunk's size where it has attention, SwiGLU experts."""
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]},
+           "shared": {"ff": z["shared_ff"]}}
+    ssm = {"type": "mamba2", "mixer": {"heads": z["ret_heads"], "vdim": z["ret_vdim"], "state": z["ret_dim"],
+                                       "groups": z["ret_heads"], "conv": 4, "norm_groups": z["ret_heads"]}}
+    diff = {"type": "attention", "mixer": {"heads": z["att_heads"], "kv_heads": z["att_kv"], "dim": z["att_dim"] // 2,
+                                           "vdim": z["att_vdim"], "scale": (z["att_dim"] // 2) ** -0.5, "diff": 0.5,
+                                           "mask": {"size": z["chunk"]}}}
+    return {"architecture": "Fakelorn", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [dict(diff if i % 4 in (0, 3) else ssm, mlp=dense if i % 4 == 0 else moe) for i in range(z["layers"])]}
+
+
+def namesun_prefill_flops(z: dict, tokens: int, like: bool = False) -> float:
+    """Multiply-adds times two of one prompt of ``tokens`` tokens as the design defines it (the recurrences as an update and
+    a read of their state per token). ``like``: of the Fakelorn arm."""
+    W, c = z["width"], z["chunk"]
+    pairs = sum(min(i + 1, c) if like else i % c + 1 for i in range(tokens))
+    H, G, D, V = z["att_heads"], z["att_kv"], z["att_dim"], z["att_vdim"]
+    Hr, Dr, Vr = z["ret_heads"], z["ret_dim"], z["ret_vdim"]
+    flops = 0.0
+    for i in range(z["layers"]):
+        if i % 4 in (0, 3):
+            per_tok = W * (H * D + G * (D + V) + H * V)
+            flops += 2.0 * pairs * H * (D + (2 if like else 1) * V)
+        else:
+            per_tok = W * (2 * Hr * Dr + 3 * Hr * Vr) + 2 * Hr * Dr * Vr
+        per_tok += 3 * W * z["ff"] if i % 4 == 0 else 3 * W * (z["top"] * z["expert_ff"] + z["shared_ff"]) + W * z["experts"]
+        flops += 2.0 * tokens * (per_tok + (2 * W * W if like else 0))
+    return flops + 2.0 * z["vocab"] * W
+
+
+def namesun_like_flops(z: dict, tokens: int) -> float:
+    return namesun_prefill_flops(z, tokens, like=True)
+
+
+def namesun_kernels(z: dict, pk: dict) -> list[dict]:
+    """Each kernel the Namesun path adds or adds an option to beside the kernel of an earlier model that does the like work,
+    on the shapes of a 2,048-token prompt portion of one sequence (or 64 decoded tokens behind 2,048 positions), L2 flushed
+    before every launch, CUDA events around one call, median of 20 (5 for the long ones). ``frac``: bytes over time
+    against the measured copy bandwidth, or flops over time against the measured bf16 rate."""
+    import torch
+
+    from tokenomos_b200 import ops
+    from tokenomos_b200.parts.registry import Runtime, builder_of
+
+    bf, dev = torch.bfloat16, "cuda"
+    T, W, P = 2048, z["width"], 16
+    flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+    rows = []
+
+    def add(name, ours_us, theirs_us, ours_work, theirs_work, unit, like):
+        peak = pk["hbm_gbs"] * 1e3 if unit == "bytes" else pk["bf16_tflops"] * 1e6       # per microsecond
+        fo, ft = ours_work / ours_us / peak, theirs_work / theirs_us / peak
+        rows.append({"kernel": name, "like": like, "unit": unit, "namesun_us": round(ours_us, 1), "namesun_frac": round(fo, 4),
+                     "like_us": round(theirs_us, 1), "like_frac": round(ft, 4), "times_further_from_roofline": round(ft / fo, 2)})
+
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    pos = torch.arange(T, dtype=torch.int32, device=dev)
+    seq = torch.zeros(T, dtype=torch.int32, device=dev)
+    cu, zero1, one1 = i32([0, T]), i32([0]), i32([1])
+
+    # 1. the stream
+    nw = torch.ones(W, device=dev)
+    res32, y = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev).to(bf)
+    add("scaled norm + residual add + the stream's rows",
+        _timed_us(lambda: ops.stream32_post_norm(res32, y, nw, 1e-6, None, 0.0, rows_out=True), flush),
+        _timed_us(lambda: ops.stream32_post_norm(res32, y, nw, 1e-6, nw, 1e-6), flush),
+        T * W * 12, T * W * 12, "bytes", "Tifisun: post-norm + residual add + norm")
+
+    # 2. attention: unit heads + value mix + cache write; prompt and decode attention over chunks
+    H, G, D, V, c = z["att_heads"], z["att_kv"], z["att_dim"], z["att_vdim"], z["chunk"]
+    pages = T // P + 1
+    pool = torch.zeros(pages, 2, G, P, max(D, V), dtype=bf, device=dev)
+    tbl = torch.arange(1, pages, dtype=torch.int32, device=dev).view(1, -1)
+    qkv = torch.randn(T, H * D + G * (D + V), device=dev).to(bf)
+    first = torch.randn(T, H * D + G * (D + V), device=dev).to(bf)[:, (H + G) * D:]
+    wq, wk = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev)
+    n = H * D + G * (D + V)
+    add("unit heads + mixed values + cache write",
+        _timed_us(lambda: ops.qkv_head_norm_write(qkv, None, None, 1e-6, pos, seq, tbl, pool, H, G, D, V, first, 0.3), flush),
+        _timed_us(lambda: ops.qkv_row_norm_write(qkv, wq, wk, 1e-6, pos, seq, tbl, pool, H, G, D, V), flush),
+        T * (n * 4 + G * V * 2), T * n * 4, "bytes", "Tifisun: query and key row norms + cache write")
+    q = ops.qkv_head_norm_write(qkv, None, None, 1e-6, pos, seq, tbl, pool, H, G, D, V)
+    pairs, windowed = sum(i % c + 1 for i in range(T)), sum(min(i + 1, c) for i in range(T))
+    scale = D ** -0.5
+    Bd = 64
+    dpos = torch.full((Bd,), T - 1, dtype=torch.int32, device=dev)
+    dseq, dtbl, dq = torch.arange(Bd, dtype=torch.int32, device=dev), tbl.expand(Bd, -1).contiguous(), q[:Bd].contiguous()
+    kv_bytes = Bd * G * min(T, c) * (D + V) * 2
+    same = D == V and ops.attention_mma_supported(H, G, D, bf)
+    out, dout = torch.empty(T, H, V, dtype=bf, device=dev), torch.empty(Bd, H, V, dtype=bf, device=dev)
+
+    def tiles(per):
+        t0 = torch.arange(0, T, per, dtype=torch.int32, device=dev)
+        return t0, torch.full_like(t0, per)
+
+    if same:
+        tc = ops.attention_prefill_tc_supported(H, G, D, bf)
+        t0, nt = tiles((ops.attention_prefill_tc_tokens if tc else ops.attention_prefill_mma_tokens)(H, G))
+        kind = "tcgen05" if tc else "mma.sync"
+
+        def prompt(reach, sink=True):
+            if tc:
+                ops.attention_prefill_tc(q, pool, out, pos, seq, tbl, t0, nt, reach, scale, None, 1, 0, sink)
+            else:
+                ops.attention_prefill_mma(q, pool, out, pos, seq, tbl, t0, nt, reach, scale, None, 0, sink)
+
+        def decode(reach):
+            ops.attention_decode_mma(dq, pool, dout, dpos, dseq, dtbl, None, reach, scale, 2, None, 0, True)
+        like = "Darizen: sliding window with a sink"
+    else:
+        t0, nt = tiles(ops.attention_biased_mma_tokens(H, G))
+        kind, like = "mma.sync", "Tifisun: sliding window with a cap and a bias"
+        bias = torch.randn(H, c, device=dev) * 0.3
+
+        def prompt(reach):
+            more = (0.0, None, True, True) if reach < 0 else (20.0, bias, True)
+            ops.attention_biased_mma(q, pool, out, pos, seq, tbl, t0, nt, None, 0, 1, reach, scale, *more)
+
+        def decode(reach):
+            more = (0.0, None, True, True) if reach < 0 else (20.0, bias, True)
+            ops.attention_biased_mma(dq, pool, dout, dpos, dseq, dtbl, None, None, None, Bd, 2, reach, scale, *more)
+
+    add(f"prompt attention over chunks with a sink ({kind})", _timed_us(lambda: prompt(-c), flush, reps=5),
+        _timed_us(lambda: prompt(c), flush, reps=5), 2.0 * pairs * H * (D + V), 2.0 * windowed * H * (D + V), "flops", like)
+    add("decode attention over chunks with a sink, 64 tokens", _timed_us(lambda: decode(-c), flush), _timed_us(lambda: decode(c), flush),
+        kv_bytes, kv_bytes, "bytes", like)
+
+    # 3. retention, beside lightning attention at equal state size
+    Hr, Dr, Vr = z["ret_heads"], z["ret_dim"], z["ret_vdim"]
+    u = torch.randn(T, 2 * Hr * Dr + 2 * Hr * Vr, device=dev).to(bf)
+    S, A = torch.zeros(66, Hr, Vr, Dr, device=dev), torch.full((Hr,), 0.99, device=dev)
+    freq = torch.rand(Dr // 2, device=dev)
+    cu64 = torch.arange(0, T + 1, T // 64, dtype=torch.int32, device=dev)
+    z64, o64 = torch.zeros(64, dtype=torch.int32, device=dev), torch.arange(1, 65, dtype=torch.int32, device=dev)
+    cu1 = torch.arange(0, 65, dtype=torch.int32, device=dev)
+
+    def retain(cu_, ctx_, slot_, n_, t=T):
+        return ops.linmem_scan(u[:t], (0, Hr * Dr, 2 * Hr * Dr), "add", "fixed", A, S, cu_, ctx_, slot_, n_, Hr, Hr, Dr, Vr,
+                               q_scale=Dr ** -0.5, freq=freq, positions=pos)
+
+    def lightning(cu_, ctx_, slot_, n_, t=T):
+        return ops.linmem_scan(u[:t], (0, Hr * Dr, 2 * Hr * Dr), "add", "fixed", A, S, cu_, ctx_, slot_, n_, Hr, Hr, Dr, Vr, act=True)
+
+    for name, a, unit, work, reps in (
+            ("2,048 tokens of one sequence", (cu, zero1, one1, 1), "flops", 4.0 * T * Hr * Dr * Vr, 5),
+            ("2,048 tokens of 64 sequences", (cu64, z64, o64, 64), "flops", 4.0 * T * Hr * Dr * Vr, 5),
+            ("one token of 64 sequences", (cu1, o64, o64, 64, 64), "bytes", 64 * Hr * Dr * Vr * 8, 20)):
+        add(f"retention: {name}", _timed_us(lambda: retain(*a), flush, reps=reps), _timed_us(lambda: lightning(*a), flush, reps=reps),
+            work, work, unit, "Tifisun: lightning attention at equal state size (32-bit)")
+    yv, inner = torch.randn(T, Hr * Vr, device=dev), Hr * Vr
+    gw = torch.ones(inner, device=dev)
+    zg = u[:, 2 * Hr * Dr + inner:]
+    add("head norm without a weight + gate", _timed_us(lambda: ops.norm_gate(yv, zg, None, 1e-6, Hr, "silu"), flush),
+        _timed_us(lambda: ops.norm_gate(yv, zg, gw, 1e-6, Hr, "silu"), flush), T * inner * 8, T * inner * 8, "bytes",
+        "Tifisun: head norm + gate")
+
+    # 4. experts
+    E, top, ff = z["experts"], z["top"], z["expert_ff"]
+    logits, corr = torch.randn(T, E, device=dev), torch.randn(E, device=dev) * 0.1
+    route_bytes = T * (E * 4 + top * 8)
+    add("routing by corrected scores among groups", _timed_us(lambda: ops.moe_route(
+        logits, E, top, 1.0, False, corr, (z["groups"], z["keep"]), False), flush),
+        _timed_us(lambda: ops.moe_route(logits, E, top, 1.0, False), flush), route_bytes, route_bytes, "bytes", "Fakelorn: routing")
+    rt = Runtime(bf, torch.device(dev))
+    # (both sides choose alike, so that both read the same experts' weights)
+    t = {"router": torch.randn(E, W, device=dev) * 0.02}
+    for e in range(E):
+        t.update({f"e{e}.gate": torch.randn(ff, W, device=dev).to(bf) * 0.02, f"e{e}.up": torch.randn(ff, W, device=dev).to(bf) * 0.02,
+                  f"e{e}.down": torch.randn(W, ff, device=dev).to(bf) * 0.02})
+    for k, shape in (("gate", (z["shared_ff"], W)), ("up", (z["shared_ff"], W)), ("down", (W, z["shared_ff"]))):
+        t["shared." + k] = torch.randn(shape, device=dev).to(bf) * 0.02
+    clamped = builder_of("feed_forward", "clamped_moe")(
+        {"experts": E, "top": top, "renorm": False, "limit": 7.0, "shared_limit": 7.0, "alpha": 1.702, "shift": 1.0}, t, rt)
+    swiglu = builder_of("feed_forward", "swiglu_moe")({"experts": E, "top": top}, t, rt)
+    for m in (T, 64, 8):
+        x = torch.randn(m, W, device=dev).to(bf)
+        flops = 6.0 * m * W * (top * ff + z["shared_ff"])
+        nbytes = 6.0 * W * (min(E, m * top) * ff + z["shared_ff"])
+        add(f"experts and shared expert, {m} tokens", _timed_us(lambda: clamped.forward(x), flush, reps=10),
+            _timed_us(lambda: swiglu.forward(x), flush, reps=10), flops if m == T else nbytes, flops if m == T else nbytes,
+            "flops" if m == T else "bytes", "Fakelorn: SwiGLU experts and shared expert")
+    return rows
+
+
 def run_design(name: str, args, warmup: int) -> int:
     """``--design darizen``: decode (batch 8 and 64) and prefill (2,048 tokens) throughput of
     Darizen stacks at a few real layer sizes, beside the LFM3 stack of sliding-window attention
@@ -2062,7 +2282,7 @@ def run_design(name: str, args, warmup: int) -> int:
 
     pk = peaks()
     sizes = {"laposun": LAPOSUN_SIZES, "lisorax": LISORAX_SIZES, "fakelorn": FAKELORN_SIZES,
-             "tifisun": TIFISUN_SIZES}.get(name, DESIGN_SIZES)
+             "tifisun": TIFISUN_SIZES, "namesun": NAMESUN_SIZES}.get(name, DESIGN_SIZES)
     for size, z in sizes.items():
         if getattr(args, "design_size", None) and size != args.design_size:
             continue
@@ -2076,6 +2296,8 @@ def run_design(name: str, args, warmup: int) -> int:
             arms = (("fakelorn", fakelorn_config(z)), ("laposun", laposun_config(z)))
         elif name == "tifisun":
             arms = (("tifisun", tifisun_config(z)), ("fakelorn", tifisun_like_config(z)))
+        elif name == "namesun":
+            arms = (("namesun", namesun_config(z)), ("fakelorn", namesun_like_config(z)))
         else:
             arms = (("darizen", darizen_config(z)), ("lfm3", lfm3_like_config(z)))
         for arm, config in arms:
@@ -2083,12 +2305,13 @@ def run_design(name: str, args, warmup: int) -> int:
                 folder = Path(tmp) / arm
                 if arm != "lfm3":
                     write_model_folder(folder, config, 0, 0.02, 0.0, torch.bfloat16)
-                    if arm == "lisorax":
-                        # the distance bias takes the logarithm of 1 + r2 * distance: its numbers are not negative
+                    if arm in ("lisorax", "namesun"):
+                        # the distance bias takes the logarithm of 1 + r2 * distance: its numbers are not negative; a
+                        # random correction of the router would send every token to the same few experts
                         from safetensors.torch import load_file, save_file
                         tensors = load_file(str(folder / "model.safetensors"))
-                        save_file({k: (v.abs() if k.endswith((".r1", ".r2")) else v) for k, v in tensors.items()},
-                                  str(folder / "model.safetensors"))
+                        save_file({k: (v.abs() if k.endswith((".r1", ".r2")) else v * 0 if k.endswith(".correction") else v)
+                                   for k, v in tensors.items()}, str(folder / "model.safetensors"))
                 else:
                     write_folder(folder, z["layers"], config)
                 model = models.load(str(folder), "cuda", models.configure(str(folder), work="bf16"))
@@ -2100,7 +2323,8 @@ def run_design(name: str, args, warmup: int) -> int:
                                            "launches": d["launches_per_step"]}
             pf = device_prefill(model, cfg, args.page)
             flops = {"laposun": laposun_prefill_flops, "lisorax": lisorax_prefill_flops, "tifisun": tifisun_prefill_flops,
-                     "fakelorn": tifisun_like_flops if name == "tifisun" else fakelorn_prefill_flops}.get(
+                     "namesun": namesun_prefill_flops,
+                     "fakelorn": {"tifisun": tifisun_like_flops, "namesun": namesun_like_flops}.get(name, fakelorn_prefill_flops)}.get(
                 arm, lambda *_: pf["flops"])(z, pf["tokens"])
             res["prefill_2048"] = {"tok_s": round(pf["tok_s"], 1), "ms": round(pf["ms"], 3),
                                    "frac": round(flops / (pf["ms"] * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)}
@@ -2108,7 +2332,7 @@ def run_design(name: str, args, warmup: int) -> int:
             del model
             torch.cuda.empty_cache()
         line["kernels"] = {"laposun": laposun_kernels, "lisorax": lisorax_kernels, "fakelorn": fakelorn_kernels,
-                           "tifisun": tifisun_kernels}.get(
+                           "tifisun": tifisun_kernels, "namesun": namesun_kernels}.get(
             name, design_kernels)(z, pk)
         print(json.dumps(line), flush=True)
     return 0
@@ -2138,9 +2362,9 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points")
     ap.add_argument("--trace", default=None,
                     help="--workload: write one JSON record per step of an extra pass to this file")
-    ap.add_argument("--design", default=None, choices=["darizen", "laposun", "lisorax", "fakelorn", "tifisun"],
+    ap.add_argument("--design", default=None, choices=["darizen", "laposun", "lisorax", "fakelorn", "tifisun", "namesun"],
                     help="the named design beside the closest existing model at equal sizes instead (darizen beside "
-                         "LFM3, laposun beside darizen, lisorax beside laposun, fakelorn beside laposun, tifisun beside fakelorn)")
+                         "LFM3, laposun beside darizen, lisorax beside laposun, fakelorn beside laposun, tifisun and namesun beside fakelorn)")
     ap.add_argument("--design-size", default=None, help="only this size of the design's table")
     ap.add_argument("--sweep", action="store_true",
                     help="decode and prefill at other batch sizes and context lengths instead")

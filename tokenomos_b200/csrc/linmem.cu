@@ -156,39 +156,46 @@ __device__ __forceinline__ float lm_step(float2 (&S)[R / 2], const float* k, con
 }
 
 // A warp stages one token's k and q (silu, rotation, unit length, q_scale), k . q and the decay per channel. A lane holds
-// the elements lane + 32 j. cs: cos and sin of the token's angles (null: no rotation).
+// the elements lane + 32 j.
 template <typename T, int DPL>
-__device__ __forceinline__ void lm_fetch(const LinMem& m, int row, int h, int lane, const float2* cs, float (&kv)[DPL],
-                                         float (&qv)[DPL]) {
+__device__ __forceinline__ void lm_fetch(const LinMem& m, int row, int h, int lane, float (&kv)[DPL], float (&qv)[DPL]) {
     const T* src = (const T*)m.qkv + (size_t)row * m.stride;
     const int kh = h / (m.H / m.K);
-    if (cs != nullptr) {
-        // (an element's partner may be another lane's: read once more)
-        auto at = [&](int off, int d) {
-            const float x = to_f<T>(src[off + kh * m.D + d]);
-            return m.act ? lm_silu(x) : x;
-        };
-#pragma unroll
-        for (int j = 0; j < DPL; ++j) {
-            const int d = lane + 32 * j;
-            kv[j] = d < m.D ? at(m.k_off, d) : 0.f;
-            qv[j] = d < m.D ? at(m.q_off, d) : 0.f;
-            if (d < 2 * m.half) {
-                const bool low = d < m.half;
-                const int other = low ? d + m.half : d - m.half;
-                const float2 c = cs[low ? d : other];
-                const float s = low ? -c.y : c.y;
-                kv[j] = kv[j] * c.x + at(m.k_off, other) * s;
-                qv[j] = qv[j] * c.x + at(m.q_off, other) * s;
-            }
-        }
-        return;
-    }
 #pragma unroll
     for (int j = 0; j < DPL; ++j) {
         const int d = lane + 32 * j;
         kv[j] = d < m.D ? to_f<T>(src[m.k_off + kh * m.D + d]) : 0.f;
         qv[j] = d < m.D ? to_f<T>(src[m.q_off + kh * m.D + d]) : 0.f;
+    }
+}
+// The same elements' partners in the rotation (which may be another lane's elements), asked for with them; and the rotation,
+// cs holding cos and sin of the token's angles.
+template <typename T, int DPL>
+__device__ __forceinline__ void lm_fetch_partners(const LinMem& m, int row, int h, int lane, float (&kp)[DPL], float (&qp)[DPL]) {
+    const T* src = (const T*)m.qkv + (size_t)row * m.stride + (size_t)(h / (m.H / m.K)) * m.D;
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+        const int d = lane + 32 * j, other = d < m.half ? d + m.half : d - m.half;
+        kp[j] = d < 2 * m.half ? to_f<T>(src[m.k_off + other]) : 0.f;
+        qp[j] = d < 2 * m.half ? to_f<T>(src[m.q_off + other]) : 0.f;
+    }
+}
+template <int DPL>
+__device__ __forceinline__ void lm_rotate(const LinMem& m, int lane, const float2* cs, float (&kv)[DPL], float (&qv)[DPL],
+                                          float (&kp)[DPL], float (&qp)[DPL]) {
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+        const int d = lane + 32 * j;
+        if (m.act) {
+            kv[j] = lm_silu(kv[j]), kp[j] = lm_silu(kp[j]);
+            qv[j] = lm_silu(qv[j]), qp[j] = lm_silu(qp[j]);
+        }
+        if (d < 2 * m.half) {
+            const float2 c = cs[d < m.half ? d : d - m.half];
+            const float s = d < m.half ? -c.y : c.y;
+            kv[j] = kv[j] * c.x + kp[j] * s;
+            qv[j] = qv[j] * c.x + qp[j] * s;
+        }
     }
 }
 template <int DPL>
@@ -253,7 +260,12 @@ linmem_prepare_kernel(const LinMem m, const LinMemPrep p) {
     for (int kh = warp; kh < m.K; kh += 8) {
         float kv[DPL], qv[DPL];
         float* dst = p.kq + ((size_t)kh * p.rows + t) * 2 * DP;
-        lm_fetch<T, DPL>(m, t, kh * (m.H / m.K), lane, m.freq != nullptr ? cs : nullptr, kv, qv);
+        lm_fetch<T, DPL>(m, t, kh * (m.H / m.K), lane, kv, qv);
+        if (m.freq != nullptr) {
+            float kp[DPL], qp[DPL];
+            lm_fetch_partners<T, DPL>(m, t, kh * (m.H / m.K), lane, kp, qp);
+            lm_rotate<DPL>(m, lane, cs, kv, qv, kp, qp);
+        }
         lm_shape<DPL>(m, lane, kv, qv, dst, dst + DP, kq_s + kh);
     }
     const T* v = (const T*)m.qkv + (size_t)t * m.stride + m.v_off;
@@ -400,7 +412,8 @@ linmem_token_kernel(const LinMem m) {
     if (len <= 0) return;
     const int r = lane & 7;
     const float A = m.A[h];
-    const bool carried = m.seq_ctx[s] > 0;
+    const int ctx = m.seq_ctx[s];
+    const bool carried = ctx > 0;
     float* st = m.state + ((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[s]) * m.H + h) * m.V * m.D;
     float2 S[CPT][R / 2];
 #pragma unroll
@@ -422,12 +435,15 @@ linmem_token_kernel(const LinMem m) {
         if (t > 0) __syncthreads();
         if (warp == 0) {
             float kv[DPL], qv[DPL];
+            lm_fetch<T, DPL>(m, row, h, lane, kv, qv);
             if (m.freq != nullptr) {
-                const float pos = (float)m.positions[row];
+                float kp[DPL], qp[DPL];
+                lm_fetch_partners<T, DPL>(m, row, h, lane, kp, qp);
+                const float pos = (float)(ctx + t);          // (the angles are formed while the loads are in flight)
                 for (int i = lane; i < m.half; i += 32) sincosf(pos * m.freq[i], &cs[i].y, &cs[i].x);
                 __syncwarp();
+                lm_rotate<DPL>(m, lane, cs, kv, qv, kp, qp);
             }
-            lm_fetch<T, DPL>(m, row, h, lane, m.freq != nullptr ? cs : nullptr, kv, qv);
             lm_shape<DPL>(m, lane, kv, qv, ks, qs, &kq_s);
         }
         if constexpr (DECAY == LM_CHANNEL) {
