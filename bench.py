@@ -398,6 +398,7 @@ def kernel_case(name: str) -> None:
     tiles of 16 tokens), 20 launches in a CUDA graph that is replayed five times;
     ``ssd_scan``: the state-space scan over a 2,048-token portion of one sequence, 4 launches;
     ``linmem_scan``: the delta rule (a decay per head) over such a portion, 4 launches of its two kernels;
+    ``retention_scan``: the same for retention (16 heads, q and k rotated);
     ``attn_portions`` (a measurement, not a profiler case): the tcgen05 prefill attention on
     portions behind cached contexts, with a tile's keys shared by 1 to 16 CTAs."""
     import torch
@@ -464,6 +465,16 @@ def kernel_case(name: str) -> None:
         for _ in range(4):
             ops.linmem_scan(u, (0, K * D, 2 * K * D), "delta", "head", vec + 1, S, i32([0, T]), i32([0]), i32([1]), 1, H, K, D, V,
                             D ** -0.5, unit=True, beta=z, gates=z[:, H:], bias=vec)
+        torch.cuda.synchronize()
+    elif name == "retention_scan":
+        T, H, D, V = 2048, 16, 128, 128
+        u = torch.randn(T, 2 * H * (D + V), device=dev).to(bf16)
+        S, A, freq = torch.zeros(2, H, V, D, device=dev), torch.full((H,), 0.99, device=dev), torch.rand(D // 2, device=dev)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        pos = torch.arange(T, dtype=torch.int32, device=dev)
+        for _ in range(4):
+            ops.linmem_scan(u, (0, H * D, 2 * H * D), "add", "fixed", A, S, i32([0, T]), i32([0]), i32([1]), 1, H, H, D, V,
+                            q_scale=D ** -0.5, freq=freq, positions=pos)
         torch.cuda.synchronize()
     elif name == "gemm_tc64":
         ws = [torch.randn(6144, 2048, device=dev, dtype=bf16) * 0.02 for _ in range(8)]
@@ -2349,7 +2360,7 @@ def main() -> int:
     ap.add_argument("--profile", default=None, choices=["decode", "decode_graph", "prefill", "ingraph"],
                     help="run only a small case for a profiler (see profile_case) and exit; ingraph: "
                          "the cost of each kind of kernel inside the captured decode step (ingraph_table)")
-    ap.add_argument("--kernel", default=None, choices=["gemm_tc64", "conv_tile", "attn_portions", "ssd_scan", "linmem_scan"],
+    ap.add_argument("--kernel", default=None, choices=["gemm_tc64", "conv_tile", "attn_portions", "ssd_scan", "linmem_scan", "retention_scan"],
                     help="run only one kernel over rotating operands for a profiler (see kernel_case) and exit")
     ap.add_argument("--ctx", type=int, default=2048, help="--profile: positions already cached")
     ap.add_argument("--gpus", type=int, default=1)

@@ -507,6 +507,25 @@ def test_retention_reads_by_distance_over_hundreds_of_tokens(dtype, tmp_path):
         close(got, {"a": want}, 1e-4 if dtype == "float32" else 4e-2, "far write")
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("case", [dict(dim=8, vdim=12, decay=[0.5, 0.99, 1.0], rot_dims=8), dict(dim=40, vdim=33, decay=[0.999, 0.95], rot_dims=8),
+                                  dict(dim=100, vdim=70, decay=[0.9995], rot_dims=66, base=1e6),
+                                  dict(dim=130, vdim=9, decay=[0.98], rot_dims=None)])
+def test_retention_over_long_portions_walked_in_segments(case, dtype, tmp_path):
+    """Portions long enough to be walked in segments side by side: whole segments and a rest, one token more than a segment,
+    beside short portions and single tokens, from zeros and from a carried state, heads that soon forget and never."""
+    rig = rig_for([dict(retention(**case), mlp=None)], 40, dtype, tmp_path, seed=13, page=16, pages=260, slots=4)
+    mixer, m = rig.model.blocks[0].mixer, rig.config["layers"][0]["mixer"]
+    lengths = {"a": 1024, "b": 1300, "c": 700, "d": 515, "e": 800}
+    plans = {"a": [(0, 1024)], "b": [(0, 3), (3, 772), (772, 1029), (1029, 1030), (1030, 1300)], "c": [(0, 513), (513, 514), (514, 700)],
+             "d": [(0, 1), (1, 515)], "e": [(0, 256), (256, 768), (768, 800)]}
+    x = rows_for(lengths, 40, 7)
+    want = {rid: plain.retention(x[rid], rig.w, "l0.mix.", m, 1e-5) for rid in x}
+    got = rig.run(x, plans, lambda rows, ctx: mixer.forward(rows, ctx, 0), live=4)
+    close(got, want, 1e-4 if dtype == "float32" else 4e-2, f"segments {case} {dtype}")
+
+
 ROUTES = [dict(E=6, top=2, groups=(3, 2)), dict(E=12, top=3, groups=(3, 1)), dict(E=5, top=5, groups=None), dict(E=40, top=8, groups=(8, 3)),
           dict(E=64, top=1, groups=(64, 2)), dict(E=96, top=6, groups=(2, 1)), dict(E=33, top=32, groups=None), dict(E=1, top=1, groups=(1, 1)),
           dict(E=128, top=4, groups=(4, 4))]

@@ -17,7 +17,12 @@
 // over the rows, (aS)^T k and (aS)^T q, run side by side and only the first is on the path from token to token.
 //
 // A step continues from the stored S exactly where the step before left it, and a token's arithmetic is the same
-// wherever the request was cut; a sequence at position 0 starts from zeros whatever its state row holds.
+// wherever the request was cut, to rounding; a sequence at position 0 starts from zeros whatever its state row holds.
+//
+// The additive rule with a fixed decay is linear in S, so a long portion need not be walked by one block per columns from
+// end to end: it is cut into segments of LM_SEG tokens, a first pass walks all of them but the last side by side for what
+// each adds to the state (no read-out), and in the second pass a segment's block starts from S' = a^LM_SEG S + (what the
+// segment before added), formed over the segments before it, all in 32-bit like the walk itself.
 #include <math.h>
 
 #include "common.cuh"
@@ -27,6 +32,7 @@ enum : int { TK_K_LINMEM = 13 };
 constexpr int LM_COLS = 4;       // columns of a warp (times the columns per thread)
 constexpr int LM_TOK = 16;       // tokens of a stage
 constexpr int LM_STAGES = 3;
+constexpr int LM_SEG = 256;      // tokens of a segment (whole stages)
 
 enum : int { LM_ADD = 0, LM_DELTA = 1 };
 enum : int { LM_FIXED = 0, LM_HEAD = 1, LM_CHANNEL = 2 };
@@ -240,7 +246,33 @@ struct LinMemPrep {
     float *kq, *g, *v;
     float4* sc;
     int rows, VP;            // T', the values' padded size
+    float* seg;              // [slots][H][V][D]: what each segment adds to the state, or null: no segments
+    int n_seqs;
 };
+
+// The segment a block works on: sequence s's segments have the slots cu_seqlens[s] / LM_SEG + s and up (as many as it can
+// need), so that the slots of all sequences together are at most tokens / LM_SEG + n_seqs.
+struct LmSegment {
+    int s, j, n;             // sequence, which of its n segments (j >= n: none)
+    int slot0;               // its first segment's slot
+};
+__device__ __forceinline__ LmSegment lm_segment(const LinMem& m, int n_seqs, int slot) {
+    // the last sequence whose first slot is not past this one (every warp looks for itself, 32 sequences at a time)
+    int lo = -1;
+    for (int s0 = 0; s0 < n_seqs; s0 += 32) {
+        const int s = s0 + (threadIdx.x & 31);
+        const unsigned before = __ballot_sync(0xffffffffu, s < n_seqs && m.cu_seqlens[s] / LM_SEG + s <= slot);
+        lo += __popc(before);
+        if (before != 0xffffffffu) break;
+    }
+    LmSegment g;
+    g.s = lo;
+    const int first = m.cu_seqlens[lo];
+    g.slot0 = first / LM_SEG + lo;
+    g.j = slot - g.slot0;
+    g.n = (m.cu_seqlens[lo + 1] - first + LM_SEG - 1) / LM_SEG;
+    return g;
+}
 
 template <typename T, int DPL, int RULE, int DECAY>
 __global__ void __launch_bounds__(256)
@@ -294,9 +326,92 @@ __device__ __forceinline__ void lm_copy16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
+// Segments, first pass: what a segment adds to the state (the sequence's first one: on top of the stored state, of which it
+// leaves a copy in the last segment's slot, since the last segment's block will overwrite the stored one).
+template <int R, int CPT>
+__global__ void __launch_bounds__(256)
+linmem_segment_kernel(const LinMem m, const LinMemPrep p) {
+    constexpr int DP = 8 * R;
+    extern __shared__ __align__(16) float smem[];        // [stage][k per token, values]
+    pdl_launch_dependents();
+    pdl_wait();
+    const LmSegment g = lm_segment(m, p.n_seqs, blockIdx.z);
+    if (g.j >= g.n - 1) return;                          // the last segment is nobody's past
+    const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.y, cols = LM_COLS * CPT * warps, c0 = blockIdx.x * cols;
+    const int first = m.cu_seqlens[g.s] + g.j * LM_SEG;
+    const int r = lane & 7, wc = warp * LM_COLS * CPT + (lane >> 3);
+    const int stage_floats = LM_TOK * (DP + cols);
+    const float* k = p.kq + ((size_t)(h / (m.H / m.K)) * p.rows + first) * 2 * DP;
+    const float* v = p.v + ((size_t)h * p.rows + first) * p.VP + c0;
+    const int v_cols = min(cols, p.VP - c0);
+    auto issue = [&](int t0, int b) {
+        if (t0 < LM_SEG) {
+            float* dst = smem + (size_t)b * stage_floats;
+            for (int i = threadIdx.x; i < LM_TOK * DP / 4; i += blockDim.x) {
+                const int t = i / (DP / 4), d = (i % (DP / 4)) * 4;
+                lm_copy16(dst + t * DP + d, k + (size_t)(t0 + t) * 2 * DP + d);
+            }
+            dst += LM_TOK * DP;
+            for (int i = threadIdx.x; i < LM_TOK * cols / 4; i += blockDim.x) {
+                const int t = i / (cols / 4), c = (i % (cols / 4)) * 4;
+                if (c < v_cols) lm_copy16(dst + t * cols + c, v + (size_t)(t0 + t) * p.VP + c);
+            }
+        }
+        asm volatile("cp.async.commit_group;\n" ::);
+    };
+#pragma unroll
+    for (int i = 0; i < LM_STAGES - 1; ++i) issue(i * LM_TOK, i);
+
+    const size_t head = (size_t)m.V * m.D;
+    const float* st = m.state + ((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[g.s]) * m.H + h) * head;
+    float* mine = p.seg + ((size_t)blockIdx.z * m.H + h) * head;
+    float* last = p.seg + ((size_t)(g.slot0 + g.n - 1) * m.H + h) * head;
+    const bool carried = m.seq_ctx[g.s] > 0 && g.j == 0;
+    float2 S[CPT][R / 2];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const int col = c0 + wc + LM_COLS * c;
+        lm_load<R>(S[c], st + (size_t)col * m.D, r, m.D, carried && col < m.V);
+        if (g.j == 0) lm_store<R>(S[c], last + (size_t)col * m.D, r, m.D, col < m.V);
+    }
+    const float2 a = two(m.A[h]);
+    int b = 0;
+    for (int t0 = 0; t0 < LM_SEG; t0 += LM_TOK) {
+        asm volatile("cp.async.wait_group %0;\n" ::"n"(LM_STAGES - 2));
+        __syncthreads();                                 // the stage is there, and the one before it is read
+        issue(t0 + (LM_STAGES - 1) * LM_TOK, (b + LM_STAGES - 1) % LM_STAGES);
+        const float* ks = smem + (size_t)b * stage_floats + 4 * r;
+        const float* vt = smem + (size_t)b * stage_floats + LM_TOK * DP + wc;
+        b = (b + 1) % LM_STAGES;
+#pragma unroll 4
+        for (int t = 0; t < LM_TOK; ++t) {
+            float2 kk[R / 2];
+#pragma unroll
+            for (int i = 0; i < R / 4; ++i) {
+                const float4 k4 = *reinterpret_cast<const float4*>(ks + t * DP + 32 * i);
+                kk[2 * i] = make_float2(k4.x, k4.y);
+                kk[2 * i + 1] = make_float2(k4.z, k4.w);
+            }
+#pragma unroll
+            for (int c = 0; c < CPT; ++c) {
+                const float2 u = two(vt[t * cols + LM_COLS * c]);
+#pragma unroll
+                for (int i = 0; i < R / 2; ++i) S[c][i] = fma2(kk[i], u, mul2(a, S[c][i]));
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;\n" ::);
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+        const int col = c0 + wc + LM_COLS * c;
+        lm_store<R>(S[c], mine + (size_t)col * m.D, r, m.D, col < m.V);
+    }
+}
+
 // Portions, second kernel: a block owns LM_COLS * CPT columns a warp of a head of a sequence and walks the sequence's
-// tokens; stages of LM_TOK tokens are copied LM_STAGES - 1 ahead.
-template <int R, int RULE, int DECAY, int CPT>
+// tokens; stages of LM_TOK tokens are copied LM_STAGES - 1 ahead. SEG: it walks one segment of the sequence.
+template <int R, int RULE, int DECAY, int CPT, bool SEG>
 __global__ void __launch_bounds__(256)
 linmem_scan_kernel(const LinMem m, const LinMemPrep p) {
     constexpr int DP = 8 * R;                            // the key size, padded
@@ -305,8 +420,14 @@ linmem_scan_kernel(const LinMem m, const LinMemPrep p) {
     pdl_launch_dependents();
     pdl_wait();
     const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int s = blockIdx.z, h = blockIdx.y, cols = LM_COLS * CPT * warps, c0 = blockIdx.x * cols;
-    const int first = m.cu_seqlens[s], len = m.cu_seqlens[s + 1] - first;
+    LmSegment sg{(int)blockIdx.z, 0, 1, 0};
+    if constexpr (SEG) {
+        sg = lm_segment(m, p.n_seqs, blockIdx.z);
+        if (sg.j >= sg.n) return;
+    }
+    const int s = sg.s, h = blockIdx.y, cols = LM_COLS * CPT * warps, c0 = blockIdx.x * cols;
+    const int first = m.cu_seqlens[s] + sg.j * LM_SEG, rest = m.cu_seqlens[s + 1] - first;
+    const int len = SEG ? min(rest, LM_SEG) : rest;
     if (len <= 0) return;
     const int r = lane & 7, wc = warp * LM_COLS * CPT + (lane >> 3);        // this thread's first column of the block
     const int stage_floats = LM_TOK * (VEC * DP + cols + 4);
@@ -339,10 +460,32 @@ linmem_scan_kernel(const LinMem m, const LinMemPrep p) {
     float* st = m.state + ((size_t)TK_SLOT(TK_K_LINMEM, m.seq_slot[s]) * m.H + h) * m.V * m.D;
     float2 S[CPT][R / 2];
     const bool carried = m.seq_ctx[s] > 0;
+    if (SEG && sg.n > 1) {
+        const size_t head = (size_t)m.V * m.D, slot = m.H * head;
+        const float* seg = p.seg + (size_t)sg.slot0 * slot + h * head;
+        const float* from = seg + (size_t)(sg.j == 0 ? sg.n - 1 : 0) * slot;     // the stored state's copy, or the first segment's
+        const float2 a = two(powf(m.A[h], (float)LM_SEG));
 #pragma unroll
-    for (int c = 0; c < CPT; ++c) {
-        const int col = c0 + wc + LM_COLS * c;
-        lm_load<R>(S[c], st + (size_t)col * m.D, r, m.D, carried && col < m.V);
+        for (int c = 0; c < CPT; ++c) {
+            const int col = c0 + wc + LM_COLS * c;
+            lm_load<R>(S[c], from + (size_t)col * m.D, r, m.D, col < m.V);
+        }
+        for (int i = 1; i < sg.j; ++i) {
+#pragma unroll
+            for (int c = 0; c < CPT; ++c) {
+                float2 more[R / 2];
+                const int col = c0 + wc + LM_COLS * c;
+                lm_load<R>(more, seg + (size_t)i * slot + (size_t)col * m.D, r, m.D, col < m.V);
+#pragma unroll
+                for (int e = 0; e < R / 2; ++e) S[c][e] = fma2(a, S[c][e], more[e]);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+            const int col = c0 + wc + LM_COLS * c;
+            lm_load<R>(S[c], st + (size_t)col * m.D, r, m.D, carried && col < m.V);
+        }
     }
     const int HV = m.H * m.V;
     float* y = m.y + (size_t)first * HV + h * m.V + c0 + wc;
@@ -388,6 +531,7 @@ linmem_scan_kernel(const LinMem m, const LinMemPrep p) {
         }
     }
     asm volatile("cp.async.wait_group 0;\n" ::);
+    if (SEG && sg.j + 1 < sg.n) return;                  // the sequence's last segment leaves the new state
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
         const int col = c0 + wc + LM_COLS * c;
@@ -397,13 +541,14 @@ linmem_scan_kernel(const LinMem m, const LinMemPrep p) {
 
 // Steps of single tokens (a few a sequence at most): the state streams through, CPT columns a thread, so that many
 // bytes are in flight; the block's warps stage a token's vectors together.
-template <typename T, int R, int RULE, int DECAY, int CPT>
-__global__ void __launch_bounds__(256)
+// (ROT: the angles' code would take registers that the state's loads in flight want: three blocks an SM)
+template <typename T, int R, int RULE, int DECAY, int CPT, bool ROT>
+__global__ void __launch_bounds__(256, ROT && R <= 16 ? 3 : 0)
 linmem_token_kernel(const LinMem m) {
     constexpr int DPL = R / 4, DP = 8 * R;
     __shared__ __align__(16) float ks[DP], qs[DP], gs[DECAY == LM_CHANNEL ? DP : 4];
     __shared__ float kq_s;
-    __shared__ float2 cs[DP / 2];
+    __shared__ float2 cs[ROT ? DP / 2 : 1];
     pdl_launch_dependents();
     pdl_wait();
     const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -436,7 +581,7 @@ linmem_token_kernel(const LinMem m) {
         if (warp == 0) {
             float kv[DPL], qv[DPL];
             lm_fetch<T, DPL>(m, row, h, lane, kv, qv);
-            if (m.freq != nullptr) {
+            if constexpr (ROT) {
                 float kp[DPL], qp[DPL];
                 lm_fetch_partners<T, DPL>(m, row, h, lane, kp, qp);
                 const float pos = (float)(ctx + t);          // (the angles are formed while the loads are in flight)
@@ -470,6 +615,16 @@ linmem_token_kernel(const LinMem m) {
 }
 
 namespace {
+// Slots of the segments of a step (0: no segments): where the additive rule would otherwise leave most of the GPU idle, or
+// might, for all that a recorded step knows of its sequences' lengths.
+int lm_slots(int tokens, int n_seqs, int H, int D, int V, int decay, int sm_count) {
+    if (decay != LM_FIXED || tokens < 2 * LM_SEG || n_seqs <= 0) return 0;
+    const int64_t cols = LM_COLS * (D > 128 ? 1 : 2) * 4, blocks = (V + cols - 1) / cols * H * n_seqs;
+    const int64_t slots = tokens / LM_SEG + n_seqs;
+    if (blocks >= 2 * sm_count && tokens > 4096) return 0;
+    return slots * H * V * D * 4 <= (int64_t)256 << 20 && slots <= 65535 ? (int)slots : 0;
+}
+
 template <typename T, int R, int RULE, int DECAY>
 void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_count, cudaStream_t stream) {
     if (scratch == nullptr) {
@@ -478,7 +633,11 @@ void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_c
         int warps = (m.V + per_warp - 1) / per_warp;
         const int blocks = (warps + 7) / 8;
         warps = (warps + blocks - 1) / blocks;
-        tk_launch(linmem_token_kernel<T, R, RULE, DECAY, CPT>, dim3(blocks, m.H, n_seqs), dim3(32 * warps), 0, stream, m);
+        const dim3 grid(blocks, m.H, n_seqs), block(32 * warps);
+        if (DECAY == LM_FIXED && m.freq != nullptr)
+            tk_launch(linmem_token_kernel<T, R, RULE, DECAY, CPT, DECAY == LM_FIXED>, grid, block, 0, stream, m);
+        else
+            tk_launch(linmem_token_kernel<T, R, RULE, DECAY, CPT, false>, grid, block, 0, stream, m);
         return;
     }
     constexpr int DP = 8 * R, VEC = DECAY == LM_CHANNEL ? 3 : 2;
@@ -489,6 +648,8 @@ void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_c
     p.v = p.kq + (size_t)m.K * p.rows * 2 * DP;
     p.sc = reinterpret_cast<float4*>(p.v + (size_t)m.H * p.rows * p.VP);
     p.g = reinterpret_cast<float*>(p.sc + (size_t)m.H * p.rows);
+    p.seg = nullptr;
+    p.n_seqs = n_seqs;
     tk_launch(linmem_prepare_kernel<T, R / 4, RULE, DECAY>, dim3(tokens), dim3(256),
               (m.K + 2 * m.half) * sizeof(float), stream, m, p);
     // Two columns a thread (one where a column alone is 32 registers) in blocks of four warps; eight warps, which share
@@ -499,12 +660,36 @@ void lm_launch(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_c
     while (warps > 1 && m.V <= LM_COLS * CPT * warps / 2) warps /= 2;
     const int cols = LM_COLS * CPT * warps;
     const size_t smem = (size_t)LM_STAGES * LM_TOK * (VEC * DP + cols + 4) * sizeof(float);
+    if constexpr (DECAY == LM_FIXED) {
+        const int slots = lm_slots(tokens, n_seqs, m.H, m.D, m.V, DECAY, sm_count);
+        if (slots > 0) {
+            // (four columns of 16 registers a thread: half the reads of shared memory per multiply-add, and segments enough)
+            constexpr int SC = R >= 32 ? 1 : R == 16 ? 4 : 2;
+            int sw = 4;
+            while (sw > 1 && m.V <= LM_COLS * SC * sw / 2) sw /= 2;
+            const int sc = LM_COLS * SC * sw;
+            const size_t sm = (size_t)LM_STAGES * LM_TOK * (VEC * DP + sc + 4) * sizeof(float);
+            p.seg = p.g;                                     // (a fixed decay stages none per channel)
+            const dim3 grid((m.V + sc - 1) / sc, m.H, slots);
+            static size_t raised_seg = 48 * 1024;
+            if (sm > raised_seg) {
+                cudaFuncSetAttribute(linmem_segment_kernel<R, SC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+                cudaFuncSetAttribute(linmem_scan_kernel<R, RULE, DECAY, SC, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                     (int)sm);
+                raised_seg = sm;
+            }
+            tk_launch_after(linmem_segment_kernel<R, SC>, grid, dim3(32 * sw),
+                            (size_t)LM_STAGES * LM_TOK * (DP + sc) * sizeof(float), stream, m, p);
+            tk_launch_after(linmem_scan_kernel<R, RULE, DECAY, SC, true>, grid, dim3(32 * sw), sm, stream, m, p);
+            return;
+        }
+    }
     static size_t raised = 48 * 1024;
     if (smem > raised) {
-        cudaFuncSetAttribute(linmem_scan_kernel<R, RULE, DECAY, CPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(linmem_scan_kernel<R, RULE, DECAY, CPT, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         raised = smem;
     }
-    tk_launch_after(linmem_scan_kernel<R, RULE, DECAY, CPT>, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * warps), smem,
+    tk_launch_after(linmem_scan_kernel<R, RULE, DECAY, CPT, false>, dim3((m.V + cols - 1) / cols, m.H, n_seqs), dim3(32 * warps), smem,
                     stream, m, p);
 }
 
@@ -520,11 +705,12 @@ void lm_rows(const LinMem& m, int n_seqs, int tokens, float* scratch, int sm_cou
 TK_API int tk_linmem_max_dim() { return 256; }
 
 // Scratch memory of a step, in units of 32 floats: none for single tokens (a few a sequence at most), else what the
-// walk's vectors take.
-TK_API int tk_linmem_scratch(int tokens, int n_seqs, int H, int K, int D, int V, int decay) {
+// walk's vectors (and the segments' states) take.
+TK_API int tk_linmem_scratch(int tokens, int n_seqs, int H, int K, int D, int V, int decay, int sm_count) {
     if (tokens < 4 * n_seqs || n_seqs == 0) return 0;
     const int64_t DP = D <= 32 ? 32 : D <= 64 ? 64 : D <= 128 ? 128 : 256, VP = (V + 3) / 4 * 4;
-    const int64_t floats = (int64_t)(tokens + LM_TOK) * (2 * K * DP + H * (VP + 4) + (decay == LM_CHANNEL ? H * DP : 0));
+    const int64_t floats = (int64_t)(tokens + LM_TOK) * (2 * K * DP + H * (VP + 4) + (decay == LM_CHANNEL ? H * DP : 0)) +
+                           (int64_t)lm_slots(tokens, n_seqs, H, D, V, decay, sm_count) * H * V * D;
     return (int)((floats + 31) / 32);
 }
 
@@ -547,10 +733,11 @@ TK_API int tk_linmem_scan(const void* qkv, int64_t stride, int q_off, int k_off,
     TK_CHECK_ARG(half >= 0 && 2 * half <= D && (half == 0 || positions != nullptr), "linear memory: %d rotated columns of %d",
                  2 * half, D);
     if (half == 0) freq = nullptr;
+    TK_CHECK_ARG(freq == nullptr || decay == LM_FIXED, "linear memory: a rotation is built for a fixed decay");
     if (n_seqs == 0) return 0;
     const LinMem m{qkv, stride, q_off, k_off, v_off, zb, zb_stride, za, za_stride, bias, A, state, cu_seqlens, seq_ctx,
                    seq_slot, y, H, K, D, V, q_scale, unit, act, freq, half, positions};
-    TK_CHECK_ARG((scratch != nullptr) == (tk_linmem_scratch(tokens, n_seqs, H, K, D, V, decay) > 0),
+    TK_CHECK_ARG((scratch != nullptr) == (tk_linmem_scratch(tokens, n_seqs, H, K, D, V, decay, sm_count) > 0),
                  "linear memory: a step of %d tokens in %d sequences without its scratch memory", tokens, n_seqs);
 #define TK_LM(TT)                                                                       \
     do {                                                                                \

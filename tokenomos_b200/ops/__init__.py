@@ -1600,7 +1600,7 @@ def linmem_scan(qkv: torch.Tensor, offsets: tuple, rule: str, decay: str, A: tor
             raise KernelError(f"linmem_scan: {name} is float32 [{T}, >= {need}] with contiguous columns")
     y = torch.empty(T, heads * v_dim, dtype=torch.float32, device=qkv.device)
     # a step with portions stages its vectors in memory first
-    n = _lib.call("tk_linmem_scratch", T, int(n_seqs), heads, kv_heads, dim, v_dim, LINMEM_DECAYS[decay])
+    n = _lib.call("tk_linmem_scratch", T, int(n_seqs), heads, kv_heads, dim, v_dim, LINMEM_DECAYS[decay], int(sm_count))
     scratch = torch.empty(n, 32, dtype=torch.float32, device=qkv.device) if n else None
     _lib.call("tk_linmem_scan", _ptr(qkv), qkv.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]), LINMEM_RULES[rule],
               _ptr(beta), beta.stride(0) if beta is not None else 0, LINMEM_DECAYS[decay], _ptr(gates),

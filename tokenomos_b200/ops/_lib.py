@@ -110,7 +110,7 @@ _SIGNATURES = {
     "tk_glu_gelu": [P, P, I, I, I, I, P],
     "tk_gemm_skinny_gelu": [P, L, P, L, P, P, L, I, I, I, I, P],
     "tk_linmem_max_dim": [],
-    "tk_linmem_scratch": [I, I, I, I, I, I, I],
+    "tk_linmem_scratch": [I, I, I, I, I, I, I, I],
     "tk_linmem_scan": [P, L, I, I, I, I, P, L, I, P, L, P, P, P, P, P, P, I, I, P, P, I, I, I, I, F, I, I, P, I, P, I, I, P],
     "tk_norm_gate": [P, P, L, P, F, P, I, I, I, I, I, P],
     "tk_pair_norm_mean": [P, L, P, L, P, P, F, F, P, I, I, I, P],
